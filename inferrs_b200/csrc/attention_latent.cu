@@ -12,6 +12,10 @@
 // numbers of ctx.  Scores, the softmax and the sums are float in both builds.  Keys come in ascending order from a
 // multiple of 32, so the order of every sum depends only on (pos, window, slices), never on the batch or the pages.
 //
+// A cached vector may be longer than the latent: behind its R numbers stands a key part that all heads share and that
+// carries the position (rotated before it was cached).  A head's query then has a second part of its own, which the
+// kernels rotate as they fetch it, and the score is scale * (q'_h . c_j + r_h . k_j); the sums run over the latent alone.
+//
 // With more than one slice of keys per row (long contexts in steps of few rows), every slice leaves its unscaled
 // sum, maximum and denominator in a workspace and a second kernel joins them.
 #include "common.cuh"
@@ -20,6 +24,30 @@
 #define LA_HPW 2                       // heads per warp
 #define LA_HEADS (LA_WARPS * LA_HPW)   // heads per block
 #define LA_KEYS 32
+#define LA_MOST_ROT 256                // places of a rotated part that the float form takes
+
+// The heads' rotated query parts: element (row, h, e) at q[row * q_row + h * q_head + e], e < src; the first 2 * half of
+// them turn by the row's position (number i with i + half).  `width` places of the cached vector belong to this part
+// (src or more: the rest is zeros); 0: there is no such part.
+struct LatentRot {
+    const void* q;
+    long q_row, q_head;
+    int src, half, width;
+    const float* cos_table;      // [table_rows, half]
+    const float* sin_table;
+    int table_rows;
+};
+
+template <typename T>
+__device__ __forceinline__ float latent_rot_value(const LatentRot& rot, int row, int h, int e, int pos) {
+    if (e >= rot.src) return 0.0f;
+    const T* q = reinterpret_cast<const T*>(rot.q) + (long)row * rot.q_row + (long)h * rot.q_head;
+    const float v = ib_to_float(q[e]);
+    if (e >= 2 * rot.half || pos < 0 || pos >= rot.table_rows) return v;
+    const int i = e < rot.half ? e : e - rot.half;
+    const float c = rot.cos_table[(long)pos * rot.half + i], s = rot.sin_table[(long)pos * rot.half + i];
+    return e < rot.half ? v * c - ib_to_float(q[e + rot.half]) * s : v * c + ib_to_float(q[i]) * s;
+}
 
 template <typename QT, int RPL>  // latent numbers per lane: R <= 32 * RPL
 __global__ void __launch_bounds__(32 * LA_WARPS)
@@ -27,11 +55,12 @@ latent_attention_kernel(const QT* __restrict__ q, long q_row, long q_head, const
                         const int* __restrict__ block_table, int max_pages, int page_size, int n_pages,
                         const int* __restrict__ row_request, const int* __restrict__ positions, int n_heads, int R,
                         float scale, int window, int n_slices, act_t* __restrict__ out, long o_row, long o_head,
-                        float* __restrict__ ws_acc, float* __restrict__ ws_ml) {
+                        float* __restrict__ ws_acc, float* __restrict__ ws_ml, const LatentRot rot) {
     extern __shared__ float smem[];
-    const int ldt = R + 1;                       // a lane per key reads down a column: odd stride, no conflicts
-    float* tile = smem;                          // [LA_KEYS][R + 1]
-    float* qs = smem + LA_KEYS * ldt;            // [LA_HEADS][R]
+    const int RK = R + rot.width;                // numbers of a cached vector: the latent and the rotated key part
+    const int ldt = RK | 1;                      // a lane per key reads down a column: odd stride, no conflicts
+    float* tile = smem;                          // [LA_KEYS][ldt]
+    float* qs = smem + LA_KEYS * ldt;            // [LA_HEADS][RK]
     ib_grid_dependency_sync();
     const int row = blockIdx.x, slice = blockIdx.z;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -46,9 +75,13 @@ latent_attention_kernel(const QT* __restrict__ q, long q_row, long q_head, const
     const int t0 = slice * per_slice;
     const int t1 = min(n_tiles, t0 + per_slice);
 
-    for (int i = threadIdx.x; i < LA_HEADS * R; i += blockDim.x) {
-        const int h = head0 + i / R;
-        qs[i] = h < n_heads ? ib_to_float(q[(long)row * q_row + (long)h * q_head + (i % R)]) * scale : 0.0f;
+    for (int i = threadIdx.x; i < LA_HEADS * RK; i += blockDim.x) {
+        const int h = head0 + i / RK, e = i % RK;
+        float v = 0.0f;
+        if (h < n_heads)
+            v = e < R ? ib_to_float(q[(long)row * q_row + (long)h * q_head + e])
+                      : latent_rot_value<QT>(rot, row, h, e - R, pos);
+        qs[i] = v * scale;
     }
 
     float acc[LA_HPW][RPL], m[LA_HPW], l[LA_HPW];
@@ -68,9 +101,9 @@ latent_attention_kernel(const QT* __restrict__ q, long q_row, long q_head, const
             const act_t* src = nullptr;
             if (j >= lo && j <= pos) {
                 const int page = bt[j / page_size];
-                if (page >= 0 && page < n_pages) src = plane + ((long)page * page_size + (j % page_size)) * R;
+                if (page >= 0 && page < n_pages) src = plane + ((long)page * page_size + (j % page_size)) * RK;
             }
-            for (int e = lane; e < R; e += 32) tile[jj * ldt + e] = src ? ib_to_float(src[e]) : 0.0f;
+            for (int e = lane; e < RK; e += 32) tile[jj * ldt + e] = src ? ib_to_float(src[e]) : 0.0f;
         }
         __syncthreads();
         const int j = j0 + lane;
@@ -80,12 +113,12 @@ latent_attention_kernel(const QT* __restrict__ q, long q_row, long q_head, const
         for (int a = 0; a < LA_HPW; ++a) {
             const int hl = warp * LA_HPW + a;
             if (head0 + hl >= n_heads) continue;     // uniform over the warp
-            const float* qh = qs + hl * R;
+            const float* qh = qs + hl * RK;
             float s = -INFINITY;
             if (valid) {
                 const float* cj = tile + lane * ldt;
                 float dot = 0.0f;
-                for (int e = 0; e < R; ++e) dot = fmaf(qh[e], cj[e], dot);
+                for (int e = 0; e < RK; ++e) dot = fmaf(qh[e], cj[e], dot);
                 s = dot;
             }
             const float m_new = fmaxf(m[a], ib_warp_max(s));
@@ -212,7 +245,8 @@ __device__ __forceinline__ void lm_cp_async16(void* dst, const void* src, int sr
 // row (blockIdx.x), any slices.  TT = 2: a block per tile of up to two tokens of one request, named by a tile list
 // (tile_req[i] < 0: no tile); the two tokens' queries meet every tile of latents together, so a prompt's latents
 // cross from L2 half as often and every B operand serves twice as many products.  One slice then.
-template <int NT, int TT>
+// ROT: cached vectors and queries have rot.width (a multiple of 16) more numbers, which join the scores alone.
+template <int NT, int TT, bool ROT>
 __global__ void __launch_bounds__(128)
 latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, long q_head,
                             const __nv_bfloat16* __restrict__ plane, const int* __restrict__ block_table, int max_pages,
@@ -220,8 +254,10 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
                             const int* __restrict__ positions, const int* __restrict__ tile_req,
                             const int* __restrict__ tile_row0, const int* __restrict__ q_start, int n_heads, float scale,
                             int window, int n_slices, __nv_bfloat16* __restrict__ out, long o_row, long o_head,
-                            float* __restrict__ ws_acc, float* __restrict__ ws_ml) {
-    constexpr int R = 32 * NT, LDC = R + LM_PAD, LDP = LM_KEYS + LM_PAD, MR = TT * LM_ROWS;
+                            float* __restrict__ ws_acc, float* __restrict__ ws_ml, const LatentRot rot) {
+    constexpr int R = 32 * NT, LDP = LM_KEYS + LM_PAD, MR = TT * LM_ROWS;
+    const int RK = ROT ? R + rot.width : R;              // numbers of a cached vector
+    const int LDC = RK + LM_PAD;
     extern __shared__ __align__(16) unsigned char lm_smem[];
     __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(lm_smem);          // [TT * 16][LDC]
     __nv_bfloat16* c_s = q_s + MR * LDC;                                     // [64][LDC]
@@ -258,6 +294,14 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
         const __nv_bfloat16* src = q + (long)(row + (ok ? tok : 0)) * q_row + (long)min(h, n_heads - 1) * q_head + ch * 8;
         lm_cp_async16(q_s + m * LDC + ch * 8, src, ok ? 16 : 0);
     }
+    if constexpr (ROT) {                              // their rotated parts, turned as they are fetched
+        for (int i = threadIdx.x; i < MR * rot.width; i += blockDim.x) {
+            const int m = i / rot.width, e = i % rot.width;
+            const int tok = m / LM_ROWS, h = head0 + m % LM_ROWS;
+            const bool ok = h < n_heads && tok < n_tok;
+            q_s[m * LDC + R + e] = __float2bfloat16_rn(ok ? latent_rot_value<__nv_bfloat16>(rot, row + tok, h, e, pos0 + tok) : 0.0f);
+        }
+    }
     // two threads per key: the page is looked up once per key and tile, each thread copies half of the latent
     auto load_tile = [&](int t) {
         const int jj = threadIdx.x >> 1, half = threadIdx.x & 1;
@@ -267,13 +311,15 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
         if (j >= lo0 && j <= pos_last) {
             const int page = bt[j / page_size];
             if (page >= 0 && page < n_pages) {
-                src = plane + ((long)page * page_size + (j % page_size)) * R;
+                src = plane + ((long)page * page_size + (j % page_size)) * RK;
                 bytes = 16;
             }
         }
         __nv_bfloat16* dst = c_s + jj * LDC;
 #pragma unroll
         for (int ch = half; ch < R / 8; ch += 2) lm_cp_async16(dst + ch * 8, bytes ? src + ch * 8 : src, bytes);
+        if constexpr (ROT)
+            for (int ch = R / 8 + half; ch < RK / 8; ch += 2) lm_cp_async16(dst + ch * 8, bytes ? src + ch * 8 : src, bytes);
     };
     if (t0 < t1) load_tile(t0);
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -303,15 +349,14 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
                 sc[tk][i][0] = sc[tk][i][1] = sc[tk][i][2] = sc[tk][i][3] = 0.0f;
                 sd[tk][i][0] = sd[tk][i][1] = sd[tk][i][2] = sd[tk][i][3] = 0.0f;
             }
-#pragma unroll
-        for (int ks = 0; ks < R / 16; ++ks) {
+        auto score_step = [&](int ks, bool second) {
             uint32_t b0, b1, b2, b3;
             lm_ldmatrix_x4(b0, b1, b2, b3, ct + (warp * 16 + (lane & 7) + (lane >> 4) * 8) * LDC + ks * 16 + ((lane >> 3) & 1) * 8);
 #pragma unroll
             for (int tk = 0; tk < TT; ++tk) {
                 uint32_t a0, a1, a2, a3;
                 lm_ldmatrix_x4(a0, a1, a2, a3, q_s + (tk * LM_ROWS + (lane & 15)) * LDC + ks * 16 + (lane >> 4) * 8);
-                if (ks & 1) {
+                if (second) {
                     lm_mma(sd[tk][0], a0, a1, a2, a3, b0, b1);
                     lm_mma(sd[tk][1], a0, a1, a2, a3, b2, b3);
                 } else {
@@ -319,7 +364,11 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
                     lm_mma(sc[tk][1], a0, a1, a2, a3, b2, b3);
                 }
             }
-        }
+        };
+#pragma unroll
+        for (int ks = 0; ks < R / 16; ++ks) score_step(ks, ks & 1);
+        if constexpr (ROT)
+            for (int ks = R / 16; ks < RK / 16; ++ks) score_step(ks, false);
         const int j_base = first + t * LM_KEYS + warp * 16 + 2 * (lane & 3);
 #pragma unroll
         for (int tk = 0; tk < TT; ++tk) {
@@ -450,24 +499,31 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
     }
 }
 
-static IbDeviceSet latent_mma_smem_set[2][17];
+#define LM_MOST_ROT 128                // places of a rotated part that the tensor-core form takes
+static IbDeviceSet latent_mma_smem_set[2][2][17];
 
-template <int NT, int TT>
+template <int NT, int TT, bool ROT>
 static int launch_latent_mma(const void* q, long q_row, long q_head, const void* plane, const int* block_table,
                              int max_pages, int page_size, int n_pages, const int* row_request, const int* positions,
                              const int* tile_req, const int* tile_row0, const int* q_start, int n_blocks, int n_heads,
                              float scale, int window, int n_slices, void* out, long o_row, long o_head, float* ws_acc,
-                             float* ws_ml, cudaStream_t stream) {
-    constexpr int R = 32 * NT, LDC = R + LM_PAD, LDP = LM_KEYS + LM_PAD, MR = TT * LM_ROWS;
-    const size_t smem = (size_t)(MR * LDC + LM_KEYS * LDC + MR * LDP) * 2 + 8 * MR * sizeof(float);
-    if (smem > 48 * 1024) {
-        const int e = ib_allow_dynamic_smem(latent_mma_smem_set[TT - 1][NT], latent_attention_mma_kernel<NT, TT>, smem);
+                             float* ws_ml, const LatentRot& rot, cudaStream_t stream) {
+    constexpr int R = 32 * NT, LDP = LM_KEYS + LM_PAD, MR = TT * LM_ROWS;
+    auto smem_for = [](int width) {
+        const int ldc = R + width + LM_PAD;
+        return (size_t)(MR * ldc + LM_KEYS * ldc + MR * LDP) * 2 + 8 * MR * sizeof(float);
+    };
+    const size_t smem = smem_for(ROT ? rot.width : 0);
+    const size_t smem_most = smem_for(ROT ? LM_MOST_ROT : 0);     // the permission is given once per device, for the most
+    if (smem_most > 48 * 1024) {
+        const int e = ib_allow_dynamic_smem(latent_mma_smem_set[ROT][TT - 1][NT], latent_attention_mma_kernel<NT, TT, ROT>,
+                                            smem_most);
         if (e != IB_OK) return e;
     }
     const dim3 grid(n_blocks, (n_heads + LM_ROWS - 1) / LM_ROWS, n_slices);
-    ib_launch(latent_attention_mma_kernel<NT, TT>, grid, 128, smem, stream, (const __nv_bfloat16*)q, q_row, q_head,
+    ib_launch(latent_attention_mma_kernel<NT, TT, ROT>, grid, 128, smem, stream, (const __nv_bfloat16*)q, q_row, q_head,
               (const __nv_bfloat16*)plane, block_table, max_pages, page_size, n_pages, row_request, positions, tile_req,
-              tile_row0, q_start, n_heads, scale, window, n_slices, (__nv_bfloat16*)out, o_row, o_head, ws_acc, ws_ml);
+              tile_row0, q_start, n_heads, scale, window, n_slices, (__nv_bfloat16*)out, o_row, o_head, ws_acc, ws_ml, rot);
     return ib_launch_status();
 }
 #endif  // IB_ACT_BF16
@@ -478,10 +534,12 @@ template <typename QT, int RPL>
 static int launch_latent(IbDeviceSet& set, const void* q, long q_row, long q_head, const void* plane,
                          const int* block_table, int max_pages, int page_size, int n_pages, const int* row_request,
                          const int* positions, int n_rows, int n_heads, int R, float scale, int window, int n_slices,
-                         void* out, long o_row, long o_head, float* ws_acc, float* ws_ml, cudaStream_t stream) {
-    const size_t smem = ((size_t)LA_KEYS * (R + 1) + (size_t)LA_HEADS * R) * sizeof(float);
+                         void* out, long o_row, long o_head, float* ws_acc, float* ws_ml, const LatentRot& rot,
+                         cudaStream_t stream) {
+    auto smem_for = [](int rk) { return ((size_t)LA_KEYS * (rk | 1) + (size_t)LA_HEADS * rk) * sizeof(float); };
+    const size_t smem = smem_for(R + rot.width);
     // the most that this form of the kernel can ask for: the permission is given once per device
-    const size_t smem_most = ((size_t)LA_KEYS * (32 * RPL + 1) + (size_t)LA_HEADS * 32 * RPL) * sizeof(float);
+    const size_t smem_most = smem_for(32 * RPL + LA_MOST_ROT);
     if (smem_most > 48 * 1024) {
         const int e = ib_allow_dynamic_smem(set, latent_attention_kernel<QT, RPL>, smem_most);
         if (e != IB_OK) return e;
@@ -489,12 +547,13 @@ static int launch_latent(IbDeviceSet& set, const void* q, long q_row, long q_hea
     const dim3 grid(n_rows, (n_heads + LA_HEADS - 1) / LA_HEADS, n_slices);
     ib_launch(latent_attention_kernel<QT, RPL>, grid, 32 * LA_WARPS, smem, stream, (const QT*)q, q_row, q_head,
               (const act_t*)plane, block_table, max_pages, page_size, n_pages, row_request, positions, n_heads, R, scale,
-              window, n_slices, (act_t*)out, o_row, o_head, ws_acc, ws_ml);
+              window, n_slices, (act_t*)out, o_row, o_head, ws_acc, ws_ml, rot);
     return ib_launch_status();
 }
 
 // q: element (row, h, e) at q[row * q_row + h * q_head + e], float (q_is_f32) or act_t; out likewise, act_t.
-// plane [n_pages, page_size, R] act_t.  n_slices > 1 needs ws_acc [rows * heads * n_slices * R] and
+// plane [n_pages, page_size, R + rot_width] act_t.  rot_width > 0: q_rot holds the heads' rotated parts (see LatentRot),
+// of q's type.  n_slices > 1 needs ws_acc [rows * heads * n_slices * R] and
 // ws_ml [rows * heads * n_slices * 2] floats.  tile_req, tile_row0 [n_tiles] and q_start (or null): the step's rows
 // cut into tiles of up to two tokens of one request each; the tensor-core form then takes two tokens per block.
 IB_EXPORT int ib_latent_attention(const void* q, int q_is_f32, long q_row, long q_head, const void* plane,
@@ -502,31 +561,43 @@ IB_EXPORT int ib_latent_attention(const void* q, int q_is_f32, long q_row, long 
                                   const int* row_request, const int* positions, int n_rows, int n_heads, int R,
                                   float scale, int window, int n_slices, void* out, long o_row, long o_head,
                                   float* ws_acc, float* ws_ml, const int* tile_req, const int* tile_row0,
-                                  const int* q_start, int n_tiles, cudaStream_t stream) {
+                                  const int* q_start, int n_tiles, const void* q_rot, long q_rot_row, long q_rot_head,
+                                  int rot_src, int rot_half, int rot_width, const float* cos_table,
+                                  const float* sin_table, int table_rows, cudaStream_t stream) {
     if (n_rows <= 0) return IB_OK;
     if (n_heads <= 0 || R <= 0 || page_size <= 0 || max_pages <= 0 || n_slices <= 0 || n_slices > 64 ||
         (n_slices > 1 && (ws_acc == nullptr || ws_ml == nullptr)))
         return IB_ERR_ARGUMENT;
-    if (R > 512) return IB_ERR_UNSUPPORTED;
+    if (rot_width < 0 || (rot_width > 0 && (q_rot == nullptr || rot_src < 0 || rot_src > rot_width || rot_half < 0 ||
+                                            2 * rot_half > rot_src ||
+                                            (rot_half > 0 && (cos_table == nullptr || sin_table == nullptr)))))
+        return IB_ERR_ARGUMENT;
+    if (R > 512 || rot_width > LA_MOST_ROT) return IB_ERR_UNSUPPORTED;
+    const LatentRot rot = {q_rot, q_rot_row, q_rot_head, rot_src, rot_half, rot_width, cos_table, sin_table, table_rows};
     int e = IB_OK;
 #if IB_ACT_BF16
     // bfloat16 queries and latents of a multiple of 32 numbers: the tensor cores
-    if (!q_is_f32 && R % 32 == 0 && page_size > 0 && ((uintptr_t)q % 16) == 0 && ((uintptr_t)plane % 16) == 0) {
+    if (!q_is_f32 && R % 32 == 0 && rot_width % 16 == 0 && rot_width <= LM_MOST_ROT && page_size > 0 && ((uintptr_t)q % 16) == 0 && ((uintptr_t)plane % 16) == 0) {
         // a list of tiles of up to two tokens (prompt portions, one slice): two tokens per block
         const bool pairs = tile_req != nullptr && tile_row0 != nullptr && q_start != nullptr && n_tiles > 0 && n_slices == 1;
         switch (R / 32) {
+#define IB_LATM_FORM(NT, TT, ROT, N, ...)                                                                            \
+        launch_latent_mma<NT, TT, ROT>(q, q_row, q_head, plane, block_table, max_pages, page_size, n_pages, row_request, \
+                                       positions, __VA_ARGS__, N, n_heads, scale, window, n_slices, out, o_row, o_head, \
+                                       ws_acc, ws_ml, rot, stream)
 #define IB_LATM(NT)                                                                                                  \
         case NT:                                                                                                     \
-            e = pairs ? launch_latent_mma<NT, 2>(q, q_row, q_head, plane, block_table, max_pages, page_size, n_pages, \
-                                                 row_request, positions, tile_req, tile_row0, q_start, n_tiles,      \
-                                                 n_heads, scale, window, 1, out, o_row, o_head, ws_acc, ws_ml, stream) \
-                      : launch_latent_mma<NT, 1>(q, q_row, q_head, plane, block_table, max_pages, page_size, n_pages, \
-                                                 row_request, positions, nullptr, nullptr, nullptr, n_rows, n_heads, \
-                                                 scale, window, n_slices, out, o_row, o_head, ws_acc, ws_ml, stream); \
+            if (rot_width > 0)                                                                                       \
+                e = pairs ? IB_LATM_FORM(NT, 2, true, n_tiles, tile_req, tile_row0, q_start)                         \
+                          : IB_LATM_FORM(NT, 1, true, n_rows, nullptr, nullptr, nullptr);                            \
+            else                                                                                                     \
+                e = pairs ? IB_LATM_FORM(NT, 2, false, n_tiles, tile_req, tile_row0, q_start)                        \
+                          : IB_LATM_FORM(NT, 1, false, n_rows, nullptr, nullptr, nullptr);                           \
             break;
             IB_LATM(1) IB_LATM(2) IB_LATM(3) IB_LATM(4) IB_LATM(5) IB_LATM(6) IB_LATM(7) IB_LATM(8) IB_LATM(9)
             IB_LATM(10) IB_LATM(11) IB_LATM(12) IB_LATM(13) IB_LATM(14) IB_LATM(15) IB_LATM(16)
 #undef IB_LATM
+#undef IB_LATM_FORM
             default: e = IB_ERR_UNSUPPORTED;
         }
         if (e != IB_ERR_UNSUPPORTED) {
@@ -543,7 +614,7 @@ IB_EXPORT int ib_latent_attention(const void* q, int q_is_f32, long q_row, long 
 #define IB_LAT(QT, QI, RPL, SI)                                                                                   \
     e = launch_latent<QT, RPL>(latent_smem_set[QI][SI], q, q_row, q_head, plane, block_table, max_pages, page_size, \
                                n_pages, row_request, positions, n_rows, n_heads, R, scale, window, n_slices, out,  \
-                               o_row, o_head, ws_acc, ws_ml, stream)
+                               o_row, o_head, ws_acc, ws_ml, rot, stream)
 #define IB_LAT_R(QT, QI)                                                                                          \
     do {                                                                                                          \
         if (R <= 32) IB_LAT(QT, QI, 1, 0); else if (R <= 64) IB_LAT(QT, QI, 2, 1);                                \

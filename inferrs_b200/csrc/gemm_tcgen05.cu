@@ -91,6 +91,7 @@ struct Params {
     long ldy;
     int n_tok, n_out, num_kb, y_is_f32;
     int inner;   // gated form: rows of the gate matrix; the up matrix follows it in w
+    int gelu;    // 1: y is 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))) of the product z (never with a sink)
     int tile_rows;   // rows of W that a tile covers (gated form: of each of the two matrices); the MMA's other rows are not used
     // scaled rows (null: x is used as it is): parts of the sums of squares of x's rows [n_in_parts][SSQ_LD]
     const float* in_ssq;
@@ -115,6 +116,7 @@ constexpr int SSQ_LD = 32;    // tokens per part of a list of sums of squares (t
 __device__ __forceinline__ float finish_value(const Params& p, float v, int tok, int feature, float inv, float old,
                                               float w, float& ssq) {
     v *= inv;
+    if (p.gelu) return ib_gelu_tanh(v);
     if (p.residual == nullptr) return v;
     const float s = old + __bfloat162float(__float2bfloat16_rn(v));
     p.residual[(long)tok * p.ld_res + feature] = s;
@@ -373,7 +375,8 @@ __global__ void __launch_bounds__(THREADS, (BN <= 64 ? 2 : 1)) gemm_kernel(const
                         ssq[j] = 0.0f;
                         if (tok < p.n_tok && feature_ok) {
                             const float o = BN <= 32 ? finish_value(p, v[j], tok, feature, fold[8 * SSQ_LD + c0 + j],
-                                                                    old_s[(c0 + j) % KEEP], w_sink, ssq[j]) : v[j];
+                                                                    old_s[(c0 + j) % KEEP], w_sink, ssq[j])
+                                                    : (p.gelu ? ib_gelu_tanh(v[j]) : v[j]);
                             if (p.y_is_f32) reinterpret_cast<float*>(p.y)[(long)tok * p.ldy + feature] = o;
                             else reinterpret_cast<__nv_bfloat16*>(p.y)[(long)tok * p.ldy + feature] = __float2bfloat16_rn(o);
                         }
@@ -459,8 +462,9 @@ __global__ void __launch_bounds__(THREADS, (BN <= 64 ? 2 : 1)) gemm_kernel(const
                 for (int j = 0; j < 16; ++j) {
                     const int tok = tile_t * BN + c0 + j;
                     if (tok < p.n_tok) {
-                        if (p.y_is_f32) reinterpret_cast<float*>(p.y)[(long)tok * p.ldy + feature] = sum[j];
-                        else reinterpret_cast<__nv_bfloat16*>(p.y)[(long)tok * p.ldy + feature] = __float2bfloat16_rn(sum[j]);
+                        const float o = p.gelu ? ib_gelu_tanh(sum[j]) : sum[j];
+                        if (p.y_is_f32) reinterpret_cast<float*>(p.y)[(long)tok * p.ldy + feature] = o;
+                        else reinterpret_cast<__nv_bfloat16*>(p.y)[(long)tok * p.ldy + feature] = __float2bfloat16_rn(o);
                     }
                 }
             }
@@ -632,7 +636,7 @@ struct Folded {
 };
 
 static int gemm_tn(const void* x, long ldx, const void* w, long ldw, void* y, long ldy, int y_is_f32, int n_tok,
-                   int n_out, int k, int split_k, const Folded& f, cudaStream_t stream) {
+                   int n_out, int k, int split_k, const Folded& f, cudaStream_t stream, int gelu = 0) {
     if (n_tok <= 0 || n_out <= 0) return IB_OK;
     if (k <= 0) return IB_ERR_ARGUMENT;
     // TMA wants 16-byte aligned bases and row strides
@@ -644,6 +648,7 @@ static int gemm_tn(const void* x, long ldx, const void* w, long ldw, void* y, lo
     tc::Params p;
     p.y = y; p.ldy = ldy; p.n_tok = n_tok; p.n_out = n_out; p.num_kb = (k + tc::BK - 1) / tc::BK; p.y_is_f32 = y_is_f32;
     p.inner = 0;
+    p.gelu = gelu;
     p.in_ssq = f.in_ssq; p.n_in_parts = f.n_in_parts; p.in_eps = f.in_eps; p.in_inv_width = f.in_width > 0 ? 1.0f / (float)f.in_width : 0.0f;
     p.residual = f.residual; p.ld_res = f.ld_res; p.sink_w = f.sink_w; p.sink_w_is_f32 = f.sink_w_is_f32; p.out_ssq = f.out_ssq;
     const int splits = choose_splits(n_tok, n_out, p.num_kb, bn, split_k);
@@ -668,6 +673,13 @@ IB_EXPORT int ib_gemm_tn_tcgen05(const void* x, long ldx, const void* w, long ld
                                  int n_tok, int n_out, int k, int split_k, cudaStream_t stream) {
     const Folded none = {nullptr, 0, 0.0f, 0, nullptr, 0, nullptr, 0, nullptr};
     return gemm_tn(x, ldx, w, ldw, y, ldy, y_is_f32, n_tok, n_out, k, split_k, none, stream);
+}
+
+// The same with the tanh form of gelu on the result, taken of the float32 sums: y = gelu_tanh(x w^T).
+IB_EXPORT int ib_gemm_tn_tcgen05_gelu(const void* x, long ldx, const void* w, long ldw, void* y, long ldy, int y_is_f32,
+                                      int n_tok, int n_out, int k, int split_k, cudaStream_t stream) {
+    const Folded none = {nullptr, 0, 0.0f, 0, nullptr, 0, nullptr, 0, nullptr};
+    return gemm_tn(x, ldx, w, ldw, y, ldy, y_is_f32, n_tok, n_out, k, split_k, none, stream, 1);
 }
 
 // The same with the norms around it folded in (up to 32 tokens; y bfloat16).  in_ssq (or null): x holds rows times a
@@ -708,6 +720,7 @@ IB_EXPORT int ib_gemm_swiglu_tcgen05_folded(const void* x, long ldx, const void*
     tc::Params p;
     p.y = y; p.ldy = ldy; p.n_tok = n_tok; p.n_out = inner; p.num_kb = (k + tc::BK - 1) / tc::BK; p.y_is_f32 = 0;
     p.inner = inner;
+    p.gelu = 0;
     p.in_ssq = in_ssq; p.n_in_parts = n_in_parts; p.in_eps = in_eps; p.in_inv_width = in_width > 0 ? 1.0f / (float)in_width : 0.0f;
     p.residual = nullptr; p.ld_res = 0; p.sink_w = nullptr; p.sink_w_is_f32 = 0; p.out_ssq = nullptr;
     p.tile_rows = tile_rows_for(inner, 1, 64, resident_for(bn, 1));

@@ -17,14 +17,9 @@
 __device__ __forceinline__ float sm_silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float sm_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float sm_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
-// the tanh form of gelu: 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))
-__device__ __forceinline__ float sm_gelu_tanh(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-}
-// What a gated feed-forward makes of a gate g and an up value u.  mode 0: g' sigmoid(slope g') (u' + 1) with
 // g' = min(g, limit), u' = clamp(u, -limit, limit); mode 1: gelu_tanh(g) u; mode 2: silu(g) u.
 __device__ __forceinline__ float sm_gate_value(int mode, float g, float u, float limit, float slope) {
-    if (mode == 1) return sm_gelu_tanh(g) * u;
+    if (mode == 1) return ib_gelu_tanh(g) * u;
     if (mode == 2) return sm_silu(g) * u;
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
@@ -437,6 +432,36 @@ IB_EXPORT int ib_clamped_gate(const void* gate_up, void* out, int n_rows, int in
     if (blocks > 148L * 16) blocks = 148L * 16;
     ib_launch(clamped_gate_kernel, (int)blocks, 256, 0, stream, (const act_t*)gate_up, (act_t*)out, inner, total, limit,
               slope, mode);
+    return ib_launch_status();
+}
+
+// ---------------------------------------------------------------------------
+// out[i] = gelu_tanh(z[i]) over n numbers; out may be z itself.  Sixteen bytes per thread where the sizes allow it.
+// ---------------------------------------------------------------------------
+template <bool VEC>
+__global__ void gelu_rows_kernel(const act_t* z, act_t* out, long n) {
+    ib_grid_dependency_sync();
+    for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long)gridDim.x * blockDim.x) {
+        if (VEC) {
+            SmActVec v = reinterpret_cast<const SmActVec*>(z)[i];
+#pragma unroll
+            for (int k = 0; k < SM_VEC; ++k) v.v[k] = ib_from_float<act_t>(ib_gelu_tanh(ib_to_float(v.v[k])));
+            reinterpret_cast<SmActVec*>(out)[i] = v;
+        } else {
+            out[i] = ib_from_float<act_t>(ib_gelu_tanh(ib_to_float(z[i])));
+        }
+    }
+}
+
+IB_EXPORT int ib_gelu_rows(const void* z, void* out, long n, cudaStream_t stream) {
+    if (n <= 0) return IB_OK;
+    if (z == nullptr || out == nullptr) return IB_ERR_ARGUMENT;
+    const bool vec = n % SM_VEC == 0 && sm_aligned16(z) && sm_aligned16(out);
+    const long units = vec ? n / SM_VEC : n;
+    long blocks = (units + 255) / 256;
+    if (blocks > 148L * 32) blocks = 148L * 32;
+    if (vec) ib_launch(gelu_rows_kernel<true>, (unsigned)blocks, 256, 0, stream, (const act_t*)z, (act_t*)out, units);
+    else ib_launch(gelu_rows_kernel<false>, (unsigned)blocks, 256, 0, stream, (const act_t*)z, (act_t*)out, units);
     return ib_launch_status();
 }
 

@@ -409,71 +409,116 @@ IB_EXPORT int ib_poly_norm(const void* z, const float* coef, void* out, int n_ro
 
 // ---------------------------------------------------------------------------
 // Two slices of one projection's rows, each divided by its root mean square and multiplied by a weight:
-//   the query latent  -> cq[row, :]                      (act_t, contiguous)
+//   the query latent     -> cq[row, :]                   (act_t, contiguous)
 //   the key/value latent -> the request's cache page at the row's position (absent for a layer that reads
-//                          another layer's latents)
-// proj is act_t [rows, ld]; the slices start at columns q_col and kv_col.  One block per row.
-// The cache plane is [n_pages, page_size, rank] act_t.
+//                           another layer's latents), and behind it, from place rot_at of the cached vector on, the
+//                           rot_src numbers that follow it in the projection: not normed, the first 2 * half of them
+//                           turned by position (number i with i + half); zeros fill the places between the latent
+//                           and rot_at and from rot_at + rot_src to the vector's end
+// proj is act_t [rows, ld]; the slices start at columns q_col and kv_col.  One block per row, one meeting for both sums.
+// The cache plane is [n_pages, page_size, plane_ld] act_t; the tables are float [table_rows, half].  VEC: sixteen bytes
+// per thread and access.
 // ---------------------------------------------------------------------------
-template <typename WT>
+template <typename T, int N> struct alignas(sizeof(T) * N >= 16 ? 16 : sizeof(T) * N) LatVec { T v[N]; };
+
+template <typename WT, int V>
+__device__ __forceinline__ float latent_sum_squares(const act_t* __restrict__ src, int n) {
+    float ss = 0.0f;
+    for (int j = threadIdx.x * V; j < n; j += blockDim.x * V) {
+        const LatVec<act_t, V> t = *reinterpret_cast<const LatVec<act_t, V>*>(src + j);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss = fmaf(ib_to_float(t.v[i]), ib_to_float(t.v[i]), ss);
+    }
+    return ss;
+}
+
+template <typename WT, int V>
+__device__ __forceinline__ void latent_scaled(const act_t* __restrict__ src, const WT* __restrict__ w, float inv,
+                                              act_t* __restrict__ dst, int n) {
+    for (int j = threadIdx.x * V; j < n; j += blockDim.x * V) {
+        const LatVec<act_t, V> t = *reinterpret_cast<const LatVec<act_t, V>*>(src + j);
+        const LatVec<WT, V> wv = *reinterpret_cast<const LatVec<WT, V>*>(w + j);
+        LatVec<act_t, V> o;
+#pragma unroll
+        for (int i = 0; i < V; ++i) o.v[i] = ib_from_float<act_t>(ib_to_float(t.v[i]) * inv * ib_to_float(wv.v[i]));
+        *reinterpret_cast<LatVec<act_t, V>*>(dst + j) = o;
+    }
+}
+
+template <typename WT, bool VEC>
 __global__ void latent_norm_store_kernel(const act_t* __restrict__ proj, long ld, int q_col, int q_rank,
                                          const WT* __restrict__ q_w, act_t* __restrict__ cq, int kv_col, int kv_rank,
-                                         const WT* __restrict__ kv_w, act_t* __restrict__ plane,
+                                         const WT* __restrict__ kv_w, act_t* __restrict__ plane, int plane_ld, int rot_at,
+                                         int rot_src, int half, const float* __restrict__ cos_table,
+                                         const float* __restrict__ sin_table, int table_rows,
                                          const int* __restrict__ block_table, int max_pages, int page_size, int n_pages,
                                          const int* __restrict__ row_request, const int* __restrict__ positions,
                                          float eps) {
-    __shared__ float red[32];
+    constexpr int V = VEC ? 16 / (int)sizeof(act_t) : 1;
+    __shared__ float red[64];
     ib_grid_dependency_sync();
     const int row = blockIdx.x;
     const act_t* src = proj + (long)row * ld;
-    {
-        float ss = 0.0f;
-        for (int j = threadIdx.x; j < q_rank; j += blockDim.x) {
-            const float v = ib_to_float(src[q_col + j]);
-            ss += v * v;
-        }
-        ss = ib_block_sum(ss, red);
-        const float inv = 1.0f / sqrtf(ss / (float)q_rank + eps);
-        for (int j = threadIdx.x; j < q_rank; j += blockDim.x)
-            cq[(long)row * q_rank + j] = ib_from_float<act_t>(ib_to_float(src[q_col + j]) * inv * ib_to_float(q_w[j]));
-    }
+    act_t* dst = nullptr;
+    int pos = 0;
     if (plane != nullptr) {
-        float ss = 0.0f;
-        for (int j = threadIdx.x; j < kv_rank; j += blockDim.x) {
-            const float v = ib_to_float(src[kv_col + j]);
-            ss += v * v;
+        pos = positions[row];
+        const int page = pos >= 0 ? block_table[(long)row_request[row] * max_pages + pos / page_size] : -1;
+        // a request that only pads a replayed step owns no pages
+        if (page >= 0 && page < n_pages) dst = plane + ((long)page * page_size + pos % page_size) * plane_ld;
+    }
+    float ssq = latent_sum_squares<WT, V>(src + q_col, q_rank);
+    float ssk = dst ? latent_sum_squares<WT, V>(src + kv_col, kv_rank) : 0.0f;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+    ssq = ib_warp_sum(ssq);
+    ssk = ib_warp_sum(ssk);
+    if (lane == 0) { red[warp] = ssq; red[32 + warp] = ssk; }
+    __syncthreads();
+    ssq = ib_warp_sum(lane < n_warps ? red[lane] : 0.0f);
+    ssk = ib_warp_sum(lane < n_warps ? red[32 + lane] : 0.0f);
+    latent_scaled<WT, V>(src + q_col, q_w, 1.0f / sqrtf(ssq / (float)q_rank + eps), cq + (long)row * q_rank, q_rank);
+    if (dst == nullptr) return;
+    latent_scaled<WT, V>(src + kv_col, kv_w, 1.0f / sqrtf(ssk / (float)kv_rank + eps), dst, kv_rank);
+    for (int j = kv_rank + threadIdx.x; j < rot_at; j += blockDim.x) dst[j] = ib_from_float<act_t>(0.0f);
+    const act_t* tail = src + kv_col + kv_rank;
+    for (int j = threadIdx.x; j < plane_ld - rot_at; j += blockDim.x) {
+        float v = j < rot_src ? ib_to_float(tail[j]) : 0.0f;
+        if (j < 2 * half && pos < table_rows) {
+            const int i = j < half ? j : j - half;
+            const float c = cos_table[(long)pos * half + i], s = sin_table[(long)pos * half + i];
+            v = j < half ? v * c - ib_to_float(tail[j + half]) * s : v * c + ib_to_float(tail[i]) * s;
         }
-        ss = ib_block_sum(ss, red);
-        const float inv = 1.0f / sqrtf(ss / (float)kv_rank + eps);
-        const int pos = positions[row];
-        const int page = block_table[(long)row_request[row] * max_pages + pos / page_size];
-        if (page >= 0 && page < n_pages) {          // a request that only pads a replayed step owns no pages
-            act_t* dst = plane + ((long)page * page_size + pos % page_size) * kv_rank;
-            for (int j = threadIdx.x; j < kv_rank; j += blockDim.x)
-                dst[j] = ib_from_float<act_t>(ib_to_float(src[kv_col + j]) * inv * ib_to_float(kv_w[j]));
-        }
+        dst[rot_at + j] = ib_from_float<act_t>(v);
     }
 }
 
 IB_EXPORT int ib_latent_norm_store(const void* proj, long ld, int q_col, int q_rank, const void* q_w, void* cq,
-                                   int kv_col, int kv_rank, const void* kv_w, int w_is_f32, void* plane,
-                                   const int* block_table, int max_pages, int page_size, int n_pages,
+                                   int kv_col, int kv_rank, const void* kv_w, int w_is_f32, void* plane, int plane_ld,
+                                   int rot_at, int rot_src, int half, const float* cos_table, const float* sin_table,
+                                   int table_rows, const int* block_table, int max_pages, int page_size, int n_pages,
                                    const int* row_request, const int* positions, int n_rows, float eps,
                                    cudaStream_t stream) {
     if (n_rows <= 0) return IB_OK;
     if (q_rank <= 0 || q_w == nullptr || cq == nullptr) return IB_ERR_ARGUMENT;
     if (plane != nullptr && (kv_rank <= 0 || kv_w == nullptr || block_table == nullptr || page_size <= 0 ||
-                             max_pages <= 0 || row_request == nullptr || positions == nullptr))
+                             max_pages <= 0 || row_request == nullptr || positions == nullptr || rot_at < kv_rank ||
+                             rot_src < 0 || plane_ld < rot_at + rot_src || half < 0 || 2 * half > rot_src ||
+                             (half > 0 && (cos_table == nullptr || sin_table == nullptr || table_rows <= 0))))
         return IB_ERR_ARGUMENT;
-    const int widest = q_rank > kv_rank ? q_rank : kv_rank;
-    const int threads = widest >= 1024 ? 256 : 128;
-    if (w_is_f32)
-        ib_launch(latent_norm_store_kernel<float>, n_rows, threads, 0, stream, (const act_t*)proj, ld, q_col, q_rank,
-                  (const float*)q_w, (act_t*)cq, kv_col, kv_rank, (const float*)kv_w, (act_t*)plane, block_table,
-                  max_pages, page_size, n_pages, row_request, positions, eps);
-    else
-        ib_launch(latent_norm_store_kernel<__nv_bfloat16>, n_rows, threads, 0, stream, (const act_t*)proj, ld, q_col,
-                  q_rank, (const __nv_bfloat16*)q_w, (act_t*)cq, kv_col, kv_rank, (const __nv_bfloat16*)kv_w,
-                  (act_t*)plane, block_table, max_pages, page_size, n_pages, row_request, positions, eps);
+    const int V = 16 / (int)sizeof(act_t);
+    const bool vec = ld % V == 0 && q_col % V == 0 && q_rank % V == 0 &&
+                     (((uintptr_t)proj | (uintptr_t)cq | (uintptr_t)q_w) & 15) == 0 &&
+                     (plane == nullptr || (kv_col % V == 0 && kv_rank % V == 0 && plane_ld % V == 0 &&
+                                           (((uintptr_t)plane | (uintptr_t)kv_w) & 15) == 0));
+    const int widest = (q_rank > kv_rank ? q_rank : kv_rank) / (vec ? V : 1);
+    const int threads = widest > 128 ? 256 : 128;
+#define IB_LNS(WT, VEC)                                                                                               \
+    ib_launch(latent_norm_store_kernel<WT, VEC>, n_rows, threads, 0, stream, (const act_t*)proj, ld, q_col, q_rank,   \
+              (const WT*)q_w, (act_t*)cq, kv_col, kv_rank, (const WT*)kv_w, (act_t*)plane, plane_ld, rot_at, rot_src, \
+              half, cos_table, sin_table, table_rows, block_table, max_pages, page_size, n_pages, row_request,        \
+              positions, eps)
+    if (w_is_f32) { if (vec) IB_LNS(float, true); else IB_LNS(float, false); }
+    else { if (vec) IB_LNS(__nv_bfloat16, true); else IB_LNS(__nv_bfloat16, false); }
+#undef IB_LNS
     return ib_launch_status();
 }

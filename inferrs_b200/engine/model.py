@@ -14,8 +14,8 @@ import torch
 
 from .. import kernels
 from ..cache.storage import KVNeed, StateNeed
-from ..parts.basic import Linear, NoNorm
-from ..parts.blocks import BuiltSubLayer
+from ..parts.basic import Linear, NoNorm, SandwichUpdate
+from ..parts.blocks import BuiltSubLayer, depth_planes
 from ..parts.registry import part_class
 from ..parts.spec import ModelSpec, TensorDecl
 from ..runtime import Runtime
@@ -189,6 +189,15 @@ class Model:
                 for name in _layer_tensor_names(layer):
                     if last_use[name] == i and name not in (spec.embedding, spec.lm_head):
                         weights.pop(name, None)
+        self.depth_planes = depth_planes(spec)
+        if self.depth_planes:
+            if spec.streams is not None or spec.position_table is not None or spec.embedding_norm is not None:
+                raise ModelError("averages over depth start from the plain embedding on a residual of one stream")
+            for k, e in enumerate(spec.schedule):
+                d = spec.layers[e.layer].depth_average
+                if d is None or d.results != k + 2:
+                    raise ModelError(f"schedule entry {k} runs layer {e.layer}: with averages over depth every layer "
+                                     f"averages the {k + 2} results that stand then")
         self._takes_after = ["after" in inspect.signature(b.forward).parameters for b in self.blocks]
         self.embedding_norm = None
         if spec.embedding_norm is not None:
@@ -209,7 +218,15 @@ class Model:
         """Run the step's rows through all scheduled layers; float32 logits [wanted rows, vocab]."""
         n = ctx.token_ids.shape[0]
         scale = 1.0 if self.spec.embedding_scale is None else self.spec.embedding_scale
-        if self.spec.streams is None and self.position_table is None:
+        pending = None
+        if self.depth_planes:
+            # the embedding is the first of the results that later layers look back on; the first norm reads it there
+            planes = torch.empty((self.depth_planes, n, self.spec.width), dtype=torch.float32, device=self.rt.device)
+            ctx.extra["depth_planes"] = planes
+            residual = torch.empty((n, self.spec.width), dtype=torch.float32, device=self.rt.device)
+            kernels.embedding_gather(self.embedding, ctx.token_ids, planes[0], self.rt.dtype, scale)
+            pending = SandwichUpdate(None, source=planes[0])
+        elif self.spec.streams is None and self.position_table is None:
             residual = torch.empty((n, self.spec.width), dtype=torch.float32, device=self.rt.device)
             kernels.embedding_gather(self.embedding, ctx.token_ids, residual, self.rt.dtype, scale)
         else:
@@ -223,7 +240,6 @@ class Model:
         if self.embedding_norm is not None:
             kernels.scaled_add_norm(residual, None, 1.0, self.embedding_norm[0], self.embedding_norm[1], None,
                                     self.rt.dtype)
-        pending = None
         schedule = self.spec.schedule
         for k, entry in enumerate(schedule):
             block = self.blocks[entry.layer]

@@ -81,12 +81,18 @@ _SIGNATURES = {
                           c_float, c_void_p, c_int, c_int, c_int, c_void_p],
     "ib_poly_norm": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
     "ib_latent_norm_store": [c_void_p, c_long, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p,
-                             c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p],
+                             c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,
+                             c_void_p, c_int, c_float, c_void_p],
     "ib_linear_scan": [c_int, c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_long, c_void_p, c_float, c_float,
                        c_void_p, c_long, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "ib_latent_attention": [c_void_p, c_int, c_long, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p,
                             c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_long, c_long, c_void_p, c_void_p,
-                            c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                            c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_long, c_long, c_int, c_int, c_int, c_void_p,
+                            c_void_p, c_int, c_void_p],
+    "ib_gelu_rows": [c_void_p, c_void_p, c_long, c_void_p],
+    "ib_sandwich_norm": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_long, c_int, c_void_p, c_void_p, c_void_p,
+                         c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_long,
+                         c_long, c_void_p, c_void_p, c_void_p],
     "ib_gemm_tn_simt_batched": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_long, c_long,
                                 c_long, c_int, c_long, c_long, c_long, c_void_p],
     "ib_scaled_add_norm": [c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p],
@@ -312,13 +318,42 @@ def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float, out: torch.Tensor
     _check(_core(act).ib_poly_norm(_p(z), _p(coef), _p(out), z.shape[0], z.shape[1], float(eps), _stream()), "poly_norm")
 
 
+@dataclass
+class LatentRotation:
+    """The key part behind a cached latent that carries the position: ``src`` numbers per head of a query and per
+    cached token, the first 2 ``half`` of them turned (number i with i + half) by the float32 tables [positions, half];
+    they stand from place ``at`` of a cached vector on, in ``width`` places (``src`` and then zeros)."""
+
+    at: int
+    src: int
+    width: int
+    half: int
+    cos: Optional[torch.Tensor]
+    sin: Optional[torch.Tensor]
+
+    def __post_init__(self):
+        if self.src < 0 or self.width < self.src or not 0 <= 2 * self.half <= self.src:
+            raise KernelError(f"latent rotation: {self.src} numbers in {self.width} places, {self.half} pairs")
+        if self.half:
+            for name, t in (("cos", self.cos), ("sin", self.sin)):
+                _need(t, name, (torch.float32,), 2)
+                if t.shape[1] != self.half or t.shape != self.cos.shape:
+                    raise KernelError(f"latent rotation: {name} has shape {tuple(t.shape)}, {self.half} pairs are needed")
+
+    @property
+    def table_rows(self) -> int:
+        return self.cos.shape[0] if self.half else 0
+
+
 def latent_norm_store(proj: torch.Tensor, q_col: int, q_weight: torch.Tensor, cq: torch.Tensor, kv_col: int,
                       kv_weight: Optional[torch.Tensor], plane: Optional[torch.Tensor],
                       block_table: Optional[torch.Tensor], row_request: torch.Tensor, positions: torch.Tensor,
-                      eps: float):
+                      eps: float, rot: Optional["LatentRotation"] = None):
     """Two slices of the rows of ``proj``, each divided by its root mean square and multiplied by its weight: columns
     q_col.. (as many as ``q_weight`` has) go to ``cq``; columns kv_col.. (as many as ``kv_weight`` has) go to the
-    request's page of ``plane`` [pages, page_size, rank] at the row's position (``plane`` None: no second slice)."""
+    request's page of ``plane`` [pages, page_size, rank] at the row's position (``plane`` None: no second slice).
+    ``rot``: the cached vectors are longer than the latent; the ``rot.src`` columns that follow it in ``proj`` go,
+    not normed and turned by position, to place ``rot.at`` of the cached vector, with zeros around them."""
     act = cq.dtype
     _need(proj, "proj", (act,), 2)
     _need(q_weight, "q_weight", _W, 1)
@@ -327,21 +362,25 @@ def latent_norm_store(proj: torch.Tensor, q_col: int, q_weight: torch.Tensor, cq
     q_rank = q_weight.shape[0]
     if cq.shape != (n, q_rank) or q_col < 0 or q_col + q_rank > ld:
         raise KernelError(f"latent_norm_store: proj {tuple(proj.shape)}, cq {tuple(cq.shape)}, columns {q_col}..")
-    kv_rank, page_size, n_pages, max_pages = 0, 0, 0, 0
+    kv_rank, page_size, n_pages, max_pages, plane_ld = 0, 0, 0, 0, 0
     if plane is not None:
         _need(plane, "plane", (act,), 3)
         _need(kv_weight, "kv_weight", (q_weight.dtype,), 1)
         _need(block_table, "block_table", _I, 2)
         _need(row_request, "row_request", _I, 1)
         _need(positions, "positions", _I, 1)
-        n_pages, page_size, kv_rank = plane.shape
+        n_pages, page_size, plane_ld = plane.shape
+        kv_rank = kv_weight.shape[0]
         max_pages = block_table.shape[1]
-        if kv_weight.shape[0] != kv_rank or kv_col < 0 or kv_col + kv_rank > ld:
+        at, src = (rot.at, rot.src) if rot is not None else (kv_rank, 0)
+        if (plane_ld != kv_rank if rot is None else plane_ld != rot.at + rot.width) or at < kv_rank or kv_col < 0 \
+                or kv_col + kv_rank + src > ld:
             raise KernelError(f"latent_norm_store: plane {tuple(plane.shape)}, weight {tuple(kv_weight.shape)}")
     _check(_core(act).ib_latent_norm_store(
         _p(proj), ld, q_col, q_rank, _p(q_weight), _p(cq), kv_col, kv_rank, _p(kv_weight),
-        int(q_weight.dtype == torch.float32), _p(plane), _p(block_table), max_pages, page_size, n_pages,
-        _p(row_request), _p(positions), n, float(eps), _stream()), "latent_norm_store")
+        int(q_weight.dtype == torch.float32), _p(plane), plane_ld,
+        *((rot.at, rot.src, rot.half, _p(rot.cos), _p(rot.sin), rot.table_rows) if rot is not None
+          else (kv_rank, 0, 0, None, None, 0)), _p(block_table), max_pages, page_size, n_pages, _p(row_request), _p(positions), n, float(eps), _stream()), "latent_norm_store")
 
 
 SCAN_CHANNEL_DECAY, SCAN_SCALAR_GATES, SCAN_FORGET_WRITE = 0, 1, 2
@@ -391,6 +430,7 @@ def linear_scan(mode: int, proj: torch.Tensor, q_col: int, k_col: int, v_col: in
 
 
 LATENT_TILE_TOKENS = 2      # tokens of a prompt portion that one block of the tensor-core form takes
+LATENT_TILE_KEYS = 64       # cached latents that it fetches at a time
 LATENT_SLICE_KEYS = 128     # fewest keys per slice when a row's keys are cut over several blocks
 LATENT_RESIDENT_BLOCKS = 296   # two blocks of the tensor-core form per SM
 
@@ -408,13 +448,15 @@ def latent_slices(n_rows: int, n_heads: int, max_kv_len: int) -> int:
 
 def latent_attention(q: torch.Tensor, plane: torch.Tensor, block_table: torch.Tensor, row_request: torch.Tensor,
                      positions: torch.Tensor, scale: float, window: Optional[int], out: torch.Tensor, n_slices: int = 1,
-                     tiles=None):
+                     tiles=None, q_rot: Optional[torch.Tensor] = None, rot: Optional[LatentRotation] = None):
     """Attention of every row over its request's cached latents, which serve every head as key and as value:
     out[h, r] = sum_j softmax_j(scale * q[h, r] . c_j) c_j over the visible j.  ``q`` and ``out`` are head-major
     [H, rows, R] (float32 or the activation dtype; the activation dtype), ``plane`` [pages, page_size, R].
     ``tiles`` = (tile_req, tile_row0, n_tiles, q_start): the step's rows cut into tiles of up to ``LATENT_TILE_TOKENS``
     tokens of one request each (``StepContext.attention_tiles``; -1 marks a place without a tile); with one slice the
-    tensor-core form then takes a tile per block."""
+    tensor-core form then takes a tile per block.  ``rot``: cached vectors carry a rotated key part behind the latent
+    (``plane`` [pages, page_size, rot.at + rot.width] with rot.at = R); ``q_rot`` [rows, H, rot.src] (any view with unit
+    last stride) holds the heads' query parts before the rotation, and their product joins the score."""
     act = out.dtype
     _need(q, "q", (torch.float32, act), 3)
     _need(out, "out", _W, 3)
@@ -424,10 +466,18 @@ def latent_attention(q: torch.Tensor, plane: torch.Tensor, block_table: torch.Te
     _need(positions, "positions", _I, 1)
     heads, n, rank = q.shape
     n_pages, page_size, r2 = plane.shape
-    if out.shape != q.shape or r2 != rank:
+    if out.shape != q.shape or r2 != rank + (0 if rot is None else rot.width) or (rot is not None and rot.at != rank):
         raise KernelError(f"latent_attention: q {tuple(q.shape)}, out {tuple(out.shape)}, plane {tuple(plane.shape)}")
     if rank > 512:
         raise KernelError(f"latent_attention: a latent of {rank} numbers is larger than the kernel's 512")
+    rot_args = (None, 0, 0, 0, 0, 0, None, None, 0)
+    if rot is not None:
+        if q_rot is None or q_rot.dtype != q.dtype or not q_rot.is_cuda or q_rot.shape != (n, heads, rot.src) \
+                or q_rot.stride(2) != 1:
+            raise KernelError(f"latent_attention: the rotated query parts must be [{n}, {heads}, {rot.src}] in {q.dtype} "
+                              f"with unit last stride")
+        rot_args = (_p(q_rot), q_rot.stride(0), q_rot.stride(1), rot.src, rot.half, rot.width, _p(rot.cos), _p(rot.sin),
+                    rot.table_rows)
     ws_acc = ws_ml = None
     if n_slices > 1:
         ws_acc = torch.empty((n * heads * n_slices, rank), dtype=torch.float32, device=q.device)
@@ -437,19 +487,21 @@ def latent_attention(q: torch.Tensor, plane: torch.Tensor, block_table: torch.Te
         page_size, n_pages, _p(row_request), _p(positions), n, heads, rank, float(scale), int(window) if window else 0,
         int(n_slices), _p(out), rank, n * rank, _p(ws_acc), _p(ws_ml),
         *((_p(tiles[0]), _p(tiles[1]), _p(tiles[3]), int(tiles[2])) if tiles is not None and n_slices == 1
-          else (None, None, None, 0)), _stream()), "latent_attention")
+          else (None, None, None, 0)), *rot_args, _stream()), "latent_attention")
     if n_slices > 1:
         count_launches(1)
 
 
 def batched_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act_dtype: torch.dtype):
     """out[b] = x[b] @ w[b].T for b < B: ``x`` [B, rows, K] (any view with unit last stride, so the heads of a
-    [rows, B*K] tensor are multiplied in place), ``w`` [B, M, K] and ``out`` [B, rows, M] contiguous.  True 32-bit
+    [rows, B*K] tensor are multiplied in place), ``w`` [B, M, K] contiguous, ``out`` [B, rows, M] (likewise a view with
+    unit last stride: the heads of a [rows, B*M] tensor are written in place).  True 32-bit
     products with float32 activations or weights, else the tensor cores (the vendor's batched product)."""
     if x.dim() != 3 or w.dim() != 3 or out.dim() != 3 or x.stride(2) != 1:
         raise KernelError("batched_linear: x, w and out must have three dimensions, x with unit last stride")
     _need(w, "w", _W, 3)
-    _need(out, "out", _W, 3)
+    if not out.is_cuda or out.dtype not in _W or out.stride(2) != 1:
+        raise KernelError(f"batched_linear: out must be a CUDA view in {_W} with unit last stride")
     b, n, k = x.shape
     m = w.shape[1]
     if w.shape != (b, m, k) or out.shape != (b, n, m) or not x.is_cuda:
@@ -457,7 +509,8 @@ def batched_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act_dtyp
     if act_dtype == torch.float32 or w.dtype == torch.float32 or x.dtype == torch.float32:
         code = _core(act_dtype).ib_gemm_tn_simt_batched(
             _p(x), int(x.dtype == torch.float32), _p(w), int(w.dtype == torch.float32), _p(out),
-            int(out.dtype == torch.float32), n, m, k, x.stride(1), k, m, b, x.stride(0), m * k, n * m, _stream())
+            int(out.dtype == torch.float32), n, m, k, x.stride(1), k, out.stride(1), b, x.stride(0), m * k,
+            out.stride(0), _stream())
         if code == -1:
             raise KernelError(f"batched_linear: no kernel for x {x.dtype}, w {w.dtype}, out {out.dtype}")
         _check(code, "gemm_tn_simt_batched")
@@ -493,6 +546,59 @@ def add_rms_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: 
                           f"out {tuple(out.shape)}, delta {None if delta is None else tuple(delta.shape)}")
     _check(_core(act).ib_add_rms_norm(_p(residual), _p(delta), _p(weight), int(weight.dtype == torch.float32),
                                       _p(out), _p(rows), n_out, width, float(eps), _stream()), "add_rms_norm")
+
+
+def sandwich_norm(source: torch.Tensor, delta: Optional[torch.Tensor], post: Optional[torch.Tensor], post_eps: float,
+                  weight: torch.Tensor, eps: float, out: torch.Tensor, residual: Optional[torch.Tensor] = None,
+                  planes: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
+                  result: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, conv=None):
+    """The residual of a block that norms its sub-layers' inputs and outputs, in one pass per row:
+
+    x = source + delta / rms(delta) * post (``delta`` None: x = source; ``post`` None: x = source + delta);
+    v = sum_j mix[j] planes[j] + mix[J] x (``mix`` [J + 1] None: v = x), ``planes`` [J, rows, width] float32;
+    out = v / rms(v) * weight.
+
+    x goes to ``result`` and v to ``residual`` (which may be ``source``) where they are given.  ``rows`` (int32 [W]): only
+    those rows are read and ``out`` has W rows.  ``conv`` = (weights [taps, width] float32, state or None, offset in a
+    slot, slots, row_request), only for steps in which every request brings exactly one row: out <- out + c(out) with
+    the causal convolution of :func:`causal_conv_rows`, whose kept inputs are moved on by one place."""
+    act = out.dtype
+    f32 = (torch.float32,)
+    _need(source, "source", f32, 2)
+    _need(delta, "delta", (act,), 2, optional=True)
+    _need(post, "post", f32, 1, optional=True)
+    _need(weight, "weight", _W, 1)
+    _need(out, "out", _W, 2)
+    _need(residual, "residual", f32, 2, optional=True)
+    _need(planes, "planes", f32, 3, optional=True)
+    _need(mix, "mix", f32, 1, optional=True)
+    _need(result, "result", f32, 2, optional=True)
+    _need(rows, "rows", _I, 1, optional=True)
+    n, width = source.shape
+    n_out = n if rows is None else rows.shape[0]
+    n_planes = 0 if planes is None else planes.shape[0]
+    same = [t for t in (delta, residual, result) if t is not None]
+    if out.shape != (n_out, width) or weight.shape[0] != width or any(t.shape != source.shape for t in same) \
+            or (post is not None and post.shape[0] != width) or (planes is not None and planes.shape[1:] != source.shape) \
+            or (mix is not None and mix.shape[0] != n_planes + 1):
+        raise KernelError(f"sandwich_norm: source {tuple(source.shape)}, out {tuple(out.shape)}, {n_planes} planes, "
+                          f"{0 if mix is None else mix.shape[0]} weights of the average")
+    conv_args = (None, 0, None, 0, 0, None, None)
+    if conv is not None:
+        conv_w, state, off, slots, row_request = conv
+        _need(conv_w, "conv weights", f32, 2)
+        _need(state, "state", f32, optional=True)
+        _need(slots, "slots", _I, 1)
+        _need(row_request, "row_request", _I, 1)
+        if conv_w.shape[1] != width or rows is not None or row_request.shape[0] != n \
+                or (conv_w.shape[0] > 1 and state is None):
+            raise KernelError(f"sandwich_norm: convolution weights {tuple(conv_w.shape)} for rows of {width}")
+        conv_args = (_p(conv_w), conv_w.shape[0], _p(state), 0 if state is None else state[0].numel(), int(off), _p(slots),
+                     _p(row_request))
+    _check(_core(act).ib_sandwich_norm(
+        _p(source), _p(delta), _p(post), float(post_eps), _p(planes), n * width, n_planes, _p(mix), _p(result),
+        _p(residual), _p(weight), int(weight.dtype == torch.float32), float(eps), _p(out), _p(rows), n_out, width,
+        *conv_args, _stream()), "sandwich_norm")
 
 
 def rms_norm_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor):
@@ -908,6 +1014,17 @@ def linear(x, w: torch.Tensor, out: torch.Tensor, act_dtype: torch.dtype, sink: 
     return None
 
 
+def gelu_linear(x, w: torch.Tensor, out: torch.Tensor, act_dtype: torch.dtype):
+    """out = gelu_tanh(x @ w.T).  A few bfloat16 rows run as one tcgen05 kernel that takes gelu of its float32 sums;
+    everything else as the product and the kernel over its rows."""
+    if act_dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.shape[0] <= TCGEN05_MAX_TOKENS \
+            and tcgen05_gemm_supported(x, w):
+        gemm_tn_tcgen05(x, w, out, gelu=True)
+        return
+    linear(x, w, out, act_dtype)
+    gelu_rows(out, out)
+
+
 def gated_linear(x, w_gate_up: torch.Tensor, out: torch.Tensor, act_dtype: torch.dtype):
     """out = silu(x @ gate.T) * (x @ up.T), ``w_gate_up`` [2 * inner, k] holding the gate matrix above the up
     matrix.  A few bfloat16 rows run as one tcgen05 kernel; everything else as the product and the gate kernel.
@@ -1179,6 +1296,16 @@ def clamped_gate(gate_up: torch.Tensor, out: torch.Tensor, limit: float, slope: 
         raise KernelError(f"clamped_gate: gate_up {tuple(gate_up.shape)} does not match out {tuple(out.shape)}")
     _check(_core(act).ib_clamped_gate(_p(gate_up), _p(out), n, inner, float(limit), float(slope), int(activation),
                                       _stream()), "clamped_gate")
+
+
+def gelu_rows(z: torch.Tensor, out: torch.Tensor):
+    """out = 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), element by element; ``out`` may be ``z``."""
+    act = out.dtype
+    _need(z, "z", (act,), 2)
+    _need(out, "out", _W, 2)
+    if out.shape != z.shape:
+        raise KernelError(f"gelu_rows: z {tuple(z.shape)}, out {tuple(out.shape)}")
+    _check(_core(act).ib_gelu_rows(_p(z), _p(out), z.numel(), _stream()), "gelu_rows")
 
 
 ROUTE_SOFTMAX_OF_CHOSEN, ROUTE_SIGMOID_SHARE, ROUTE_SOFTMAX_SHARE = 0, 1, 2
@@ -1847,6 +1974,8 @@ def _gemm_lib():
         lib.ib_gemm_tn_tcgen05.argtypes = [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int,
                                            c_int, c_int, c_void_p]
         lib.ib_gemm_tn_tcgen05.restype = c_int
+        lib.ib_gemm_tn_tcgen05_gelu.argtypes = lib.ib_gemm_tn_tcgen05.argtypes
+        lib.ib_gemm_tn_tcgen05_gelu.restype = c_int
         lib.ib_gemm_swiglu_tcgen05.argtypes = [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int,
                                                c_void_p]
         lib.ib_gemm_swiglu_tcgen05.restype = c_int
@@ -1898,11 +2027,13 @@ def _scaled_args(x):
     return x, (None, 0, 0.0, 0)
 
 
-def gemm_tn_tcgen05(x, w: torch.Tensor, out: torch.Tensor, split_k: int = 0, sink: Optional[ResidualSink] = None):
+def gemm_tn_tcgen05(x, w: torch.Tensor, out: torch.Tensor, split_k: int = 0, sink: Optional[ResidualSink] = None,
+                    gelu: bool = False):
     """out = x @ w.T with TMA-fed tcgen05 MMAs: W is the 128-row operand, the tokens are the N dimension.
     ``split_k`` 0 lets the kernel library choose how many CTAs of a cluster share one output tile.  ``x`` may be
     :class:`ScaledRows` and the result may go to a :class:`ResidualSink` (both: up to 32 rows, bfloat16 out); with a
-    sink the :class:`ScaledRows` that stand for the next norm's output are returned."""
+    sink the :class:`ScaledRows` that stand for the next norm's output are returned.  ``gelu``: out = gelu_tanh(x @ w.T)
+    (plain rows, no sink)."""
     xt, scaled = _scaled_args(x)
     _need(xt, "x", (torch.bfloat16,), 2)
     _need(w, "w", (torch.bfloat16,), 2)
@@ -1912,8 +2043,11 @@ def gemm_tn_tcgen05(x, w: torch.Tensor, out: torch.Tensor, split_k: int = 0, sin
     if w.shape[1] != k or out.shape != (n, m):
         raise KernelError(f"gemm: x {tuple(xt.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
     lib = _gemm_lib()
+    if gelu and (scaled[0] is not None or sink is not None):
+        raise KernelError("gemm_tn_tcgen05: gelu has no form with folded norms")
     if scaled[0] is None and sink is None:
-        code = lib.ib_gemm_tn_tcgen05(_p(xt), k, _p(w), k, _p(out), m, int(out.dtype == torch.float32), n, m, k, split_k,
+        f = lib.ib_gemm_tn_tcgen05_gelu if gelu else lib.ib_gemm_tn_tcgen05
+        code = f(_p(xt), k, _p(w), k, _p(out), m, int(out.dtype == torch.float32), n, m, k, split_k,
                                       _stream())
         if code == -1:
             raise KernelError(f"gemm_tn_tcgen05: K={k} must be a multiple of 8 and the bases 16-byte aligned")

@@ -4,3 +4,4 @@ from . import vebonex  # noqa: F401
 from . import tikizen  # noqa: F401
 from . import sefalorn  # noqa: F401
 from . import ruzunex  # noqa: F401
+from . import dasusun  # noqa: F401

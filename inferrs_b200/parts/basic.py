@@ -44,18 +44,31 @@ class StreamUpdate:
         self.delta, self.mix, self.gain = delta, mix, gain
 
 
+class SandwichUpdate:
+    """What a block that norms its sub-layers' outputs hands on: x = source + delta / rms(delta) * post, and then, with
+    an ``average`` = (planes [J, rows, width], weights [J + 1]), the weighted sum of the planes and x.  The norm kernel that
+    follows does it all (:class:`RMSNorm`).  ``source`` None: the residual itself; ``delta`` None: nothing is added;
+    ``post`` None: ``delta`` is added as it is; ``result``: where x goes before the average."""
+
+    def __init__(self, delta: Optional[torch.Tensor], post: Optional[torch.Tensor] = None, eps: float = 0.0,
+                 source: Optional[torch.Tensor] = None, average=None, result: Optional[torch.Tensor] = None):
+        self.delta, self.post, self.eps = delta, post, eps
+        self.source, self.average, self.result = source, average, result
+
+
 class RMSNorm:
     """x / sqrt(mean(x^2) + eps) * w, in float32 (inferrs-kernels/candle-kernels/src/reduce.cu:188-228),
     fused with the residual addition that precedes it in a block.  With ``groups`` > 1 every one of that many equal
     consecutive parts of the row is divided by its own root mean square.  On a residual of several streams
     [rows, streams, width] the kernel also brings the pending output into the streams and reads their weighted
-    sum (``read``; None: the plain sum)."""
+    sum (``read``; None: the plain sum).  With a ``weight_offset`` the weight is offset + the stored one, in float32."""
 
     graph_safe = True  # launches depend only on shapes, never on the step's host-side values
 
     @staticmethod
     def declare(spec: NormSpec) -> List[TensorDecl]:
-        return [TensorDecl(spec.weight, (spec.size,), init="norm")]
+        offset = getattr(spec, "weight_offset", 0.0)
+        return [TensorDecl(spec.weight, (spec.size,), init=f"uniform:{1.0 - offset}:0.1" if offset else "norm")]
 
     def __init__(self, spec: NormSpec, weights: Dict[str, torch.Tensor], rt: Runtime):
         if spec.weight is None:
@@ -63,9 +76,16 @@ class RMSNorm:
         self.spec = spec
         self.rt = rt
         self.weight = weights[spec.weight]
+        offset = getattr(spec, "weight_offset", 0.0)
+        if offset:
+            self.weight = self.weight.to(torch.float32) + offset
 
     def add_norm(self, residual: torch.Tensor, delta, rows: Optional[torch.Tensor] = None,
-                 read: Optional[torch.Tensor] = None):
+                 read: Optional[torch.Tensor] = None, conv=None):
+        """``conv``: the arguments of the convolution that follows, for a step of single rows
+        (:func:`~inferrs_b200.kernels.sandwich_norm`)."""
+        if isinstance(delta, SandwichUpdate) or conv is not None:
+            return self._sandwich(residual, delta, rows, conv)
         delta = _nothing_pending(delta)
         groups = getattr(self.spec, "groups", 1)
         if residual.dim() == 3 or groups != 1 or isinstance(delta, StreamUpdate) or read is not None:
@@ -85,6 +105,20 @@ class RMSNorm:
         n = residual.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, self.spec.size), dtype=self.rt.dtype, device=residual.device)
         kernels.add_rms_norm(residual, delta, self.weight, self.spec.eps, out, rows)
+        return out
+
+    def _sandwich(self, residual: torch.Tensor, delta, rows: Optional[torch.Tensor], conv):
+        u = delta if isinstance(delta, SandwichUpdate) else SandwichUpdate(_nothing_pending(delta))
+        if residual.dim() != 2 or getattr(self.spec, "groups", 1) != 1 or isinstance(u.delta, (StreamUpdate, kernels.ScaledRows)):
+            raise ValueError("a normed and scaled output joins the plain residual [rows, width] through a norm without groups")
+        source = residual if u.source is None else u.source
+        planes, mix = u.average if u.average is not None else (None, None)
+        moved = u.delta is not None or u.source is not None or mix is not None
+        n = residual.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((n, self.spec.size), dtype=self.rt.dtype, device=residual.device)
+        kernels.sandwich_norm(source, u.delta, u.post, u.eps, self.weight, self.spec.eps, out,
+                              residual=residual if moved and rows is None else None, planes=planes, mix=mix,
+                              result=u.result if rows is None else None, rows=rows, conv=conv)
         return out
 
     def sink(self, residual: torch.Tensor) -> "kernels.ResidualSink":

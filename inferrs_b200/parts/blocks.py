@@ -7,7 +7,7 @@ import torch
 
 from .. import kernels
 from ..cache.storage import StateNeed
-from .basic import GatedUpdate, Linear, StreamUpdate
+from .basic import GatedUpdate, Linear, SandwichUpdate, StreamUpdate
 from .registry import register_arrangement
 from .spec import TensorDecl
 
@@ -24,6 +24,10 @@ class BuiltSubLayer:
         kw = {} if sink is None else {"sink": sink}
         y = self.part.forward(ctx, cache_id, h, **kw) if self.category == "mixer" else self.part.forward(ctx, h, **kw)
         return self.post_norm.norm(y) if self.post_norm is not None else y
+
+    def run_part(self, ctx, cache_id: int, h):
+        """The part alone, without the norm on its output."""
+        return self.part.forward(ctx, cache_id, h) if self.category == "mixer" else self.part.forward(ctx, h)
 
     def takes_scaled_rows(self, n_rows: int) -> bool:
         """Whether this sub-layer can be handed scaled rows in place of its norm's output: the norm must be able to
@@ -104,6 +108,11 @@ class InputConv:
     @staticmethod
     def state_need(spec) -> Optional[StateNeed]:
         return StateNeed(shape=((spec.taps - 1) * spec.width,)) if spec.taps > 1 else None
+
+    def single_rows(self, ctx, cache_id: int):
+        """What a norm kernel needs to apply this convolution itself in a step in which every request brings one row."""
+        s = self.spec
+        return (self.weight, ctx.storage.side_state(cache_id, s) if s.taps > 1 else None, 0, ctx.slots, ctx.row_request)
 
     def __call__(self, ctx, cache_id: int, h: torch.Tensor) -> torch.Tensor:
         s = self.spec
@@ -318,3 +327,99 @@ def _width_of(sub) -> int:
 
 
 register_arrangement("gated_residual", GatedResidualBlock)
+
+
+class SandwichBlock:
+    """For every sub-layer in turn: h = norm(x), h += conv(h) (where it has an ``input_conv``), x += layer_scale *
+    post_norm(part(h)); with a ``depth_average`` the block hands on the weighted sum of the embedding and all layers'
+    results so far instead of its own result.  A sub-layer without a norm on its output adds it as it is.
+
+    As in :class:`SequentialBlock` nothing is added where a sub-layer ends: its raw output is handed on as a pending
+    :class:`~inferrs_b200.parts.basic.SandwichUpdate`, and the kernel of the norm that follows does the output's norm and
+    scale, the addition to the float32 stream, the average over depth and the norm in one pass (in steps of single rows
+    the next sub-layer's convolution too).  The results of earlier layers stand in the step's planes
+    (:func:`depth_planes`), float32.
+    """
+
+    needs_weights = True     # the model hands the arrangement the weights too: scales, averages and convolutions
+
+    @staticmethod
+    def declare(spec) -> List[TensorDecl]:
+        out = []
+        for s in spec.sublayers:
+            if s.layer_scale is not None:
+                out.append(TensorDecl(s.layer_scale, (_width_of(s),), init="uniform:1:0.3"))
+            if s.input_conv is not None:
+                out += InputConv.declare(s.input_conv)
+        if spec.depth_average is not None:
+            n = spec.depth_average.results
+            out.append(TensorDecl(spec.depth_average.weight, (n,), init=f"uniform:{1.0 / n}:{0.5 / n}"))
+        return out + [TensorDecl(name, shape) for name, shape in spec.unused]
+
+    @staticmethod
+    def side_states(spec):
+        """The inputs that the sub-layers' convolutions keep, each under its own description."""
+        needs = [(s.input_conv, InputConv.state_need(s.input_conv)) for s in spec.sublayers if s.input_conv is not None]
+        return [(owner, need) for owner, need in needs if need is not None]
+
+    def __init__(self, spec, sublayers: List[BuiltSubLayer], weights=None, rt=None):
+        if not sublayers:
+            raise ValueError("a layer needs at least one sub-layer")
+        if weights is None:
+            raise ValueError("a sandwich block needs the weights of its scales")
+        self.spec = spec
+        self.sublayers = list(sublayers)
+        self.posts, self.convs = [], []
+        for s, built in zip(spec.sublayers, sublayers):
+            if built.norm is None or not hasattr(built.norm, "add_norm") or built.sum_norm is not None:
+                raise ValueError("a sub-layer of a sandwich block has a norm before it")
+            # the norm's weight and the scale behind it are one vector, in float32
+            post, eps = None, 0.0
+            if built.post_norm is not None:
+                if getattr(built.post_norm.spec, "kind", None) != "rms" or getattr(built.post_norm.spec, "groups", 1) != 1:
+                    raise ValueError("the norm on a sub-layer's output is a plain RMS norm")
+                post, eps = built.post_norm.weight.to(torch.float32), float(built.post_norm.spec.eps)
+                if s.layer_scale is not None:
+                    post = post * weights[s.layer_scale].to(torch.float32)
+                post = post.contiguous()
+            elif s.layer_scale is not None:
+                raise ValueError("a sub-layer's scale stands behind a norm on its output")
+            self.posts.append((post, eps))
+            self.convs.append(InputConv(s.input_conv, weights) if s.input_conv is not None else None)
+        self.average = None
+        if spec.depth_average is not None:
+            self.average = weights[spec.depth_average.weight].to(torch.float32).contiguous()
+            if spec.depth_average.results < 2:
+                raise ValueError("an average over depth has the embedding and this layer's result at least")
+
+    def parts(self):
+        for s in self.sublayers:
+            yield s.part
+            yield s.norm
+            if s.post_norm is not None:
+                yield s.post_norm
+
+    def forward(self, ctx, cache_id: int, residual: torch.Tensor, pending):
+        if residual.dim() != 2:
+            raise ValueError("a sandwich block runs on the plain residual [rows, width]")
+        for s, (post, eps), conv in zip(self.sublayers, self.posts, self.convs):
+            if conv is not None and ctx.max_q_len == 1:
+                h = s.norm.add_norm(residual, pending, conv=conv.single_rows(ctx, cache_id))
+            else:
+                h = s.norm.add_norm(residual, pending)
+                if conv is not None:
+                    h = conv(ctx, cache_id, h)
+            pending = SandwichUpdate(s.run_part(ctx, cache_id, h), post, eps)
+        if self.average is not None:
+            planes, n = ctx.extra["depth_planes"], self.spec.depth_average.results - 1
+            pending.average = (planes[:n], self.average)
+            pending.result = planes[n] if n < planes.shape[0] else None      # the last result is read by nobody else
+        return pending
+
+
+def depth_planes(spec) -> int:
+    """How many results of earlier layers (the embedding among them) a model's averages over depth look back on."""
+    return max([layer.depth_average.results - 1 for layer in spec.layers if layer.depth_average is not None], default=0)
+
+
+register_arrangement("sandwich", SandwichBlock)

@@ -9,7 +9,7 @@ from .. import kernels
 from ..runtime import Runtime
 from .basic import Linear, fuse_rows
 from .registry import register_feed_forward
-from .spec import GatedDenseSpec, PolyNormDenseSpec, RoutedExpertsSpec, TensorDecl
+from .spec import DenseSpec, GatedDenseSpec, PolyNormDenseSpec, RoutedExpertsSpec, TensorDecl
 
 
 class GatedDense:
@@ -60,6 +60,33 @@ class GatedDense:
 
 
 register_feed_forward("gated_dense", GatedDense)
+
+
+class Dense:
+    """down( gelu_tanh(up(x)) ).  For a few bfloat16 rows the up product takes gelu of its float32 sums itself."""
+
+    graph_safe = True
+
+    @staticmethod
+    def declare(spec: DenseSpec) -> List[TensorDecl]:
+        return [TensorDecl(spec.up_proj, (spec.inner, spec.width)),
+                TensorDecl(spec.down_proj, (spec.width, spec.inner))]
+
+    def __init__(self, spec: DenseSpec, weights: Dict[str, torch.Tensor], rt: Runtime):
+        if spec.activation != "gelu_tanh":
+            raise ValueError(f"feed-forward without a gate: activation '{spec.activation}' has no kernel (only 'gelu_tanh')")
+        self.spec = spec
+        self.rt = rt
+        self.up = Linear(weights[spec.up_proj], rt)
+        self.down = Linear(weights[spec.down_proj], rt)
+
+    def forward(self, ctx, h):
+        a = torch.empty((h.shape[0], self.spec.inner), dtype=self.rt.dtype, device=h.device)
+        kernels.gelu_linear(h, self.up.weight, a, self.rt.dtype)
+        return self.down(a)
+
+
+register_feed_forward("dense", Dense)
 
 
 class RoutedExperts:

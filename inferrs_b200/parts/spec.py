@@ -11,7 +11,7 @@ A part's description is any frozen dataclass with a ``kind`` string; the
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Any, Optional, Tuple
 
 
@@ -34,7 +34,8 @@ class TensorDecl:
 @dataclass(frozen=True)
 class NormSpec:
     """x / sqrt(mean(x^2) + eps) * weight.  ``groups`` > 1: the row is cut into that many equal consecutive parts
-    and each part is divided by its own root mean square.  ``weight`` None (where a part allows it: the per-head
+    and each part is divided by its own root mean square.  ``weight_offset`` is added to the weight (1: the weight is
+    stored around zero and a weight of zero leaves the divided row as it is).  ``weight`` None (where a part allows it: the per-head
     norms of attention): the division alone.  ``kind="layer_norm"``: (x - mean) / sqrt(variance + eps) * weight, the
     variance being the mean of the squared deviations from the mean; no bias."""
 
@@ -43,6 +44,7 @@ class NormSpec:
     weight: Optional[str]
     kind: str = "rms"
     groups: int = 1
+    weight_offset: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -148,6 +150,19 @@ class GatedDenseSpec:
     kind: str = "gated_dense"
     limit: Optional[float] = None
     slope: float = 1.702
+
+
+@dataclass(frozen=True)
+class DenseSpec:
+    """down( act(up(x)) ), without a gate.  ``activation="gelu_tanh"``: act(z) = 0.5 z (1 + tanh(sqrt(2 / pi)
+    (z + 0.044715 z^3)))."""
+
+    width: int
+    inner: int
+    up_proj: str
+    down_proj: str
+    activation: str = "gelu_tanh"
+    kind: str = "dense"
 
 
 @dataclass(frozen=True)
@@ -382,12 +397,16 @@ class ScalarGateScanSpec:
 
 @dataclass(frozen=True)
 class LatentAttentionSpec:
-    """Attention whose keys and values are made per head from one cached latent per token, without positions.
+    """Attention whose keys and values are made per head from one cached latent per token.
 
     c_q = rmsnorm(dq(x)), q = uq(c_q) [n_heads, key_dim]; c = rmsnorm(dkv(x)) [kv_rank] is what the cache holds;
     k_h = uk_h c, v_h = uv_h c [value_dim]; scores (q . k) * scale over j <= i (``window``: i - window < j), softmax;
-    the heads times sigmoid(gate(x)) go through ``o_proj``.  ``own_kv=False``: the layer has no ``dkv`` and reads
-    the latents that another schedule entry writes."""
+    the heads times sigmoid(gate(x)) go through ``o_proj`` (``gate_proj`` None: without the gate).
+    ``own_kv=False``: the layer has no ``dkv`` and reads the latents that another schedule entry writes.
+
+    ``rot_dim`` > 0: positions.  A head's query is [key_dim, rot_dim], ``dkv`` has rot_dim more rows behind the latent's,
+    which are not normed and serve all heads as one further key part; both parts turn by ``position`` (its first
+    ``position.rot_dim`` numbers), and the score is (q . k_h + q_rot . k_rot) * scale."""
 
     width: int
     n_heads: int
@@ -402,13 +421,15 @@ class LatentAttentionSpec:
     uq_proj: str
     uk_proj: str
     uv_proj: str
-    gate_proj: str
     o_proj: str
+    gate_proj: Optional[str] = None
     dkv_proj: Optional[str] = None
     dkv_norm: Optional[str] = None
     window: Optional[int] = None
     own_kv: bool = True
     kind: str = "latent_attention"
+    rot_dim: int = 0
+    position: Optional[PositionSpec] = None
 
 
 @dataclass(frozen=True)
@@ -446,6 +467,16 @@ class ResidualGateSpec:
 
 
 @dataclass(frozen=True)
+class DepthAverageSpec:
+    """What a layer hands on is a learned average over depth: with X_0 the embedding and X_l the result of the l-th
+    layer that ran (before its own average), x <- sum_{j < results} weight[j] X_j.  ``results`` counts the embedding, the
+    layers before this one and this one.  ``weight`` names the tensor [results]."""
+
+    weight: str
+    results: int
+
+
+@dataclass(frozen=True)
 class SubLayerSpec:
     """One sub-layer of a block: a part with what stands before and after it.
 
@@ -466,6 +497,9 @@ class SubLayerSpec:
     sum_norm: Optional[Any] = None
     # a short convolution over time on what the part reads (InputConvSpec), for arrangements that apply it
     input_conv: Optional[Any] = None
+    # a vector that the part's output (after ``post_norm``) is multiplied by element by element, for arrangements that
+    # apply it: the tensor's name
+    layer_scale: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -482,11 +516,19 @@ class LayerSpec:
 
     ``arrangement="gated_residual"``: for every sub-layer in turn, h = norm(x), x += sigmoid(W h + b) * part(h), with
     W and b from the sub-layer's ``connection`` (a :class:`ResidualGateSpec`).
+
+    ``arrangement="sandwich"``: for every sub-layer in turn, h = norm(x), h += conv(h) where the sub-layer has an
+    ``input_conv``, x += layer_scale * post_norm(part(h)); and where the layer has a ``depth_average``, what it hands on
+    is that average of the results so far.
+
+    ``unused``: tensors that the weight files hold for this layer and that nothing reads, as (name, shape).
     """
 
     sublayers: Tuple[SubLayerSpec, ...]
     arrangement: str = "sequential"
     residual_scale: float = 1.0
+    depth_average: Optional[DepthAverageSpec] = None
+    unused: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()
 
     def parts_of(self, category: str) -> Tuple[Any, ...]:
         return tuple(s.part for s in self.sublayers if s.category == category)
@@ -507,13 +549,12 @@ class LayerSpec:
         for s in self.sublayers:
             if s.category == category:
                 if seen == index:
-                    s = SubLayerSpec(part=part, category=category, norm=s.norm, post_norm=s.post_norm,
-                                     connection=s.connection, sum_norm=s.sum_norm, input_conv=s.input_conv)
+                    s = replace(s, part=part)
                 seen += 1
             subs.append(s)
         if seen <= index:
             raise ValueError(f"the layer has {seen} sub-layers of category '{category}', none with index {index}")
-        return LayerSpec(sublayers=tuple(subs), arrangement=self.arrangement, residual_scale=self.residual_scale)
+        return replace(self, sublayers=tuple(subs))
 
 
 def pre_norm_layer(mixer_norm: Any, mixer: Any, ffn_norm: Any, ffn: Any) -> LayerSpec:
