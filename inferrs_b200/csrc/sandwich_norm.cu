@@ -54,8 +54,8 @@ __device__ __forceinline__ void sw_store4(float* p, const float (&d)[4]) {
 
 // The row in registers: NV groups of four columns per thread (thread t has groups t, t + blockDim, ...).  A group
 // beyond the row is read as the last one and not written, so that loads carry no condition.
-template <typename WT, int NV>
-__global__ void sandwich_norm_vec_kernel(const SandwichArgs a) {
+template <typename WT, int NV, int THREADS, bool CONV>
+__global__ void __launch_bounds__(THREADS) sandwich_norm_vec_kernel(const SandwichArgs a) {
     __shared__ float red[32];
     ib_grid_dependency_launch();
     const int W = a.width, nv = W >> 2;
@@ -73,13 +73,16 @@ __global__ void sandwich_norm_vec_kernel(const SandwichArgs a) {
     ib_grid_dependency_wait();
     const int r = blockIdx.x;
     const long src = a.rows ? a.rows[r] : r;
-    float x[NV][4], d[NV][4], v[NV][4], cv[NV][4];
+    float x[NV][4], d[NV][4], v[NV][4], cv[CONV ? NV : 1][4];
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         sw_load4(x[k], a.source + src * W + col[k]);
         if (a.delta) sw_load4(d[k], a.delta + src * W + col[k]);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) v[k][i] = cv[k][i] = 0.0f;
+        for (int i = 0; i < 4; ++i) {
+            v[k][i] = 0.0f;
+            if constexpr (CONV) cv[k][i] = 0.0f;
+        }
     }
     if (a.mix) {
         const float* p = a.planes + src * W;
@@ -96,8 +99,8 @@ __global__ void sandwich_norm_vec_kernel(const SandwichArgs a) {
         }
     }
     float* kept = nullptr;
-    if (a.conv_w && a.taps > 1) {
-        kept = a.state + (long)a.slots[a.row_request[r]] * a.slot_stride + a.state_off;
+    if constexpr (CONV) {
+        if (a.taps > 1) kept = a.state + (long)a.slots[a.row_request[r]] * a.slot_stride + a.state_off;
         for (int j = 0; j + 1 < a.taps; ++j) {
 #pragma unroll
             for (int k = 0; k < NV; ++k) {
@@ -150,7 +153,7 @@ __global__ void sandwich_norm_vec_kernel(const SandwichArgs a) {
             o.v[i] = ib_from_float<act_t>(v[k][i] * inv * w[i]);
             h[i] = ib_to_float(o.v[i]);
         }
-        if (a.conv_w) {
+        if constexpr (CONV) {
             float cw[4];
             sw_load4(cw, a.conv_w + (long)(a.taps - 1) * W + col[k]);
 #pragma unroll
@@ -220,18 +223,23 @@ static IbDeviceSet sandwich_smem_f32, sandwich_smem_bf16;
 template <typename WT>
 static int launch_sandwich(const SandwichArgs& a, int n_rows, bool vec, IbDeviceSet& set, cudaStream_t stream) {
     const int nv = a.width / 4;
-    if (vec && nv <= 4096) {
-        if (nv <= 128) ib_launch(sandwich_norm_vec_kernel<WT, 1>, n_rows, 128, 0, stream, a);
-        else if (nv <= 256) ib_launch(sandwich_norm_vec_kernel<WT, 1>, n_rows, 256, 0, stream, a);
-        else if (nv <= 512) ib_launch(sandwich_norm_vec_kernel<WT, 1>, n_rows, 512, 0, stream, a);
-        else if (nv <= 1024) ib_launch(sandwich_norm_vec_kernel<WT, 2>, n_rows, 512, 0, stream, a);
-        else if (nv <= 2048) ib_launch(sandwich_norm_vec_kernel<WT, 4>, n_rows, 512, 0, stream, a);
-        else ib_launch(sandwich_norm_vec_kernel<WT, 4>, n_rows, 1024, 0, stream, a);
+    if (vec && nv <= 2048) {
+#define IB_SANDWICH(NV, THREADS)                                                                              \
+    do {                                                                                                      \
+        if (a.conv_w) ib_launch(sandwich_norm_vec_kernel<WT, NV, THREADS, true>, n_rows, THREADS, 0, stream, a); \
+        else ib_launch(sandwich_norm_vec_kernel<WT, NV, THREADS, false>, n_rows, THREADS, 0, stream, a);      \
+    } while (0)
+        if (nv <= 128) IB_SANDWICH(1, 128);
+        else if (nv <= 256) IB_SANDWICH(1, 256);
+        else if (nv <= 512) IB_SANDWICH(1, 512);
+        else if (nv <= 1024) IB_SANDWICH(2, 512);
+        else IB_SANDWICH(4, 512);
+#undef IB_SANDWICH
         return ib_launch_status();
     }
     const size_t smem = (size_t)a.width * sizeof(float), smem_most = 200 * 1024;
     if (smem > smem_most) return IB_ERR_UNSUPPORTED;
-    if (smem > 48 * 1024) {
+    if (smem > 40 * 1024) {      // (with the static part beside it)
         const int e = ib_allow_dynamic_smem(set, sandwich_norm_kernel<WT>, smem_most);
         if (e != IB_OK) return e;
     }

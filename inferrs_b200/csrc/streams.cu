@@ -177,14 +177,14 @@ IB_EXPORT int ib_stream_add_norm(float* residual, const void* delta, const float
     if (smem > smem_most) return IB_ERR_UNSUPPORTED;
     const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
     if (weight_is_f32) {
-        if (smem > 48 * 1024) {
+        if (smem > 40 * 1024) {      // (with the static part beside it)
             const int e = ib_allow_dynamic_smem(stream_norm_smem_f32, stream_add_norm_kernel<float>, smem_most);
             if (e != IB_OK) return e;
         }
         ib_launch(stream_add_norm_kernel<float>, n_rows, threads, smem, stream, residual, (const act_t*)delta, mix, gain,
                   read, (const float*)weight, (act_t*)out, rows, streams, width, groups, eps);
     } else {
-        if (smem > 48 * 1024) {
+        if (smem > 40 * 1024) {      // (with the static part beside it)
             const int e = ib_allow_dynamic_smem(stream_norm_smem_bf16, stream_add_norm_kernel<__nv_bfloat16>, smem_most);
             if (e != IB_OK) return e;
         }

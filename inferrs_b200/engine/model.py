@@ -83,9 +83,14 @@ def check_schedule(spec: ModelSpec):
     if not spec.schedule:
         raise ModelError("the schedule is empty")
     writers: Dict[int, int] = {}
+    averages = depth_planes(spec) > 0
     for i, e in enumerate(spec.schedule):
         if not 0 <= e.layer < len(spec.layers):
             raise ModelError(f"schedule entry {i} names layer {e.layer}; the model has {len(spec.layers)}")
+        average = spec.layers[e.layer].depth_average
+        if averages and (average is None or average.results != i + 2):
+            raise ModelError(f"schedule entry {i} runs layer {e.layer}: with averages over depth every layer averages the "
+                             f"{i + 2} results that stand then")
         for mixer, cls in _mixers(spec, e.layer):
             if cls.cache_need(mixer) is None and cls.state_need(mixer) is None:
                 continue
@@ -193,11 +198,6 @@ class Model:
         if self.depth_planes:
             if spec.streams is not None or spec.position_table is not None or spec.embedding_norm is not None:
                 raise ModelError("averages over depth start from the plain embedding on a residual of one stream")
-            for k, e in enumerate(spec.schedule):
-                d = spec.layers[e.layer].depth_average
-                if d is None or d.results != k + 2:
-                    raise ModelError(f"schedule entry {k} runs layer {e.layer}: with averages over depth every layer "
-                                     f"averages the {k + 2} results that stand then")
         self._takes_after = ["after" in inspect.signature(b.forward).parameters for b in self.blocks]
         self.embedding_norm = None
         if spec.embedding_norm is not None:

@@ -334,15 +334,16 @@ class LatentRotation:
     def __post_init__(self):
         if self.src < 0 or self.width < self.src or not 0 <= 2 * self.half <= self.src:
             raise KernelError(f"latent rotation: {self.src} numbers in {self.width} places, {self.half} pairs")
-        if self.half:
-            for name, t in (("cos", self.cos), ("sin", self.sin)):
-                _need(t, name, (torch.float32,), 2)
-                if t.shape[1] != self.half or t.shape != self.cos.shape:
-                    raise KernelError(f"latent rotation: {name} has shape {tuple(t.shape)}, {self.half} pairs are needed")
 
-    @property
-    def table_rows(self) -> int:
-        return self.cos.shape[0] if self.half else 0
+    def tables(self):
+        """(cos, sin, rows) as a launch takes them."""
+        if not self.half:
+            return None, None, 0
+        for name, t in (("cos", self.cos), ("sin", self.sin)):
+            _need(t, name, (torch.float32,), 2)
+            if t.shape[1] != self.half or t.shape != self.cos.shape:
+                raise KernelError(f"latent rotation: {name} has shape {tuple(t.shape)}, {self.half} pairs are needed")
+        return _p(self.cos), _p(self.sin), self.cos.shape[0]
 
 
 def latent_norm_store(proj: torch.Tensor, q_col: int, q_weight: torch.Tensor, cq: torch.Tensor, kv_col: int,
@@ -379,7 +380,7 @@ def latent_norm_store(proj: torch.Tensor, q_col: int, q_weight: torch.Tensor, cq
     _check(_core(act).ib_latent_norm_store(
         _p(proj), ld, q_col, q_rank, _p(q_weight), _p(cq), kv_col, kv_rank, _p(kv_weight),
         int(q_weight.dtype == torch.float32), _p(plane), plane_ld,
-        *((rot.at, rot.src, rot.half, _p(rot.cos), _p(rot.sin), rot.table_rows) if rot is not None
+        *((rot.at, rot.src, rot.half, *rot.tables()) if rot is not None
           else (kv_rank, 0, 0, None, None, 0)), _p(block_table), max_pages, page_size, n_pages, _p(row_request), _p(positions), n, float(eps), _stream()), "latent_norm_store")
 
 
@@ -476,8 +477,7 @@ def latent_attention(q: torch.Tensor, plane: torch.Tensor, block_table: torch.Te
                 or q_rot.stride(2) != 1:
             raise KernelError(f"latent_attention: the rotated query parts must be [{n}, {heads}, {rot.src}] in {q.dtype} "
                               f"with unit last stride")
-        rot_args = (_p(q_rot), q_rot.stride(0), q_rot.stride(1), rot.src, rot.half, rot.width, _p(rot.cos), _p(rot.sin),
-                    rot.table_rows)
+        rot_args = (_p(q_rot), q_rot.stride(0), q_rot.stride(1), rot.src, rot.half, rot.width, *rot.tables())
     ws_acc = ws_ml = None
     if n_slices > 1:
         ws_acc = torch.empty((n * heads * n_slices, rank), dtype=torch.float32, device=q.device)
