@@ -36,6 +36,13 @@ a gelu feed-forward and routed experts) beside the Sefalorn design, the closest 
 side, window attention with a distance penalty, a matrix state in slots, routed experts), at equal width, heads,
 layers and feed-forward size, and the design's own kernels each beside the like kernel of the closest model.
 
+    python bench.py --design dasusun [--design-layers N]
+
+does the same for the Dasusun design (attention over cached latents with a rotated key part and a window, norms on both
+sides of every sub-layer, averages over depth, a short convolution in front of every mixer) beside the Vebonex design with
+latent attention in every layer, the closest existing model, at equal width, heads, latents, layers and feed-forward
+size, and the design's own kernels each beside the like kernel of the closest model.
+
     python bench.py --design sefalorn [--design-layers N]
 
 does the same for the Sefalorn design (window attention with mixed heads and a distance penalty beside the gated
@@ -280,6 +287,30 @@ def ruzunex_config(width: int, heads: int, ff: int, n_layers: int, vocab: int) -
             "canon": {"taps": 4}, "max_positions": 8192, "layers": [layer(i) for i in range(n_layers)]}
 
 
+def dasusun_config(width: int, heads: int, ff: int, q_rank: int, kv_rank: int, n_layers: int, vocab: int, positions: int,
+                   window: int) -> dict:
+    """A window in three of four layers (``window`` 0: in none), a rotated part of 64 numbers with stretched frequencies,
+    three taps in front of every mixer."""
+    def layer(i):
+        m = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": q_rank, "kv_rank": kv_rank,
+             "scale": 192 ** -0.5, "rot": {"base": 1e6, "dims": 64, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0,
+                                                                               "slow": 1.0}}}
+        if window and i % 4 != 3:
+            m["mask"] = {"size": window}
+        return {"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff}}
+    return {"architecture": "Dasusun", "vocab": vocab, "width": width, "max_positions": positions, "norm": {"eps": 1e-5},
+            "canon": {"taps": 3}, "layers": [layer(i) for i in range(n_layers)]}
+
+
+def vebonex_latent_config(width: int, heads: int, ff: int, q_rank: int, kv_rank: int, n_layers: int, vocab: int,
+                          positions: int) -> dict:
+    """Vebonex with latent attention (latents of its own) in every layer."""
+    m = {"heads": heads, "dim": 128, "vdim": 128, "q_rank": q_rank, "kv_rank": kv_rank, "scale": 128 ** -0.5}
+    return {"architecture": "Vebonex", "vocab": vocab, "width": width, "max_positions": positions, "streams": 2,
+            "norm": {"eps": 1e-5, "groups": 4},
+            "layers": [{"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff}} for _ in range(n_layers)]}
+
+
 def design_bench(args) -> int:
     import argparse as ap_
     import gc
@@ -352,6 +383,41 @@ def design_bench(args) -> int:
         r["frac_bf16"] = round(r["TFLOPs"] / pk["bf16_tflops"], 4)
         return r
 
+    if args.design == "dasusun":
+        sizes = []
+        shapes = (("width 2048", 2048, 16, 8192, 768, 512), ("width 4096", 4096, 32, 16384, 1536, 512),
+                  ("width 2048, latent 256", 2048, 16, 8192, 768, 256))
+        for name, width, heads, ff, q_rank, kv_rank in shapes:
+            n_layers = args.design_layers
+            size = (width, heads, ff, q_rank, kv_rank, n_layers, vocab, positions)
+            sizes.append({"size": name, "layers": n_layers, "heads": heads, "ff": ff, "latent": kv_rank,
+                          "dasusun": measure(dasusun_config(*size, window=1024)),
+                          "dasusun_without_windows": measure(dasusun_config(*size, window=0)),
+                          "vebonex_equal_size": measure(vebonex_latent_config(*size))})
+        rows = []
+        for heads, rank in ((16, 512), (32, 512), (16, 256)):
+            # the attention with a rotated part, without and with a window, each followed by the kernel without either
+            for form, n in (("prefill", 1), ("decode", 8), ("decode", 64)):
+                at = dict(form=form, batch=n, context=2048, tokens=2048, context_before=0, heads=heads, rank=rank, slices=0)
+                rows.append(microbench.latent(ns(rot=64, window=0, **at)))
+                rows.append(microbench.latent(ns(rot=0, window=0, **at)))
+                rows.append(microbench.latent(ns(rot=64, window=1024, **at)))
+                rows.append(microbench.latent(ns(rot=0, window=1024, **at)))
+        for n in (2048, 8):
+            for rot in (64, 0):
+                rows.append(microbench.latent_store(ns(tokens=n, q_rank=768, rank=512, rot=rot)))
+            for width in (2048, 4096):
+                for planes in (0, 4, 8):
+                    rows.append(microbench.residual(ns(impl="sandwich", tokens=n, width=width, planes=planes,
+                                                       taps=3 if n == 8 and planes else 0)))
+                for impl in ("streams", "add"):
+                    rows.append(microbench.residual(ns(impl=impl, tokens=n, width=width, planes=0, taps=0)))
+            for impl in ("gelu", "poly") if n > 16 else ("product", "plain-product", "poly"):
+                rows.append(microbench.activation(ns(impl=impl, tokens=n, inner=8192, k=2048)))
+        print(json.dumps({"design": "Dasusun", "dtype": "bf16", "data": "synthetic: seeded uniform token ids, random weights",
+                          "prompt_len": PROMPT_LEN, "decode_batch": batch, "decode_steps": args.design_steps,
+                          "peaks": pk, "sizes": sizes, "kernels": [fractions(r) for r in rows]}))
+        return 0
     if args.design == "ruzunex":
         sizes = []
         for name, width, heads, ff in (("width 2048", 2048, 16, 8192), ("width 4096", 4096, 32, 16384)):
@@ -508,7 +574,7 @@ def main() -> int:
     ap.add_argument("--clock-interval-ms", type=int, default=200, help="how often nvidia-smi is asked for the clocks")
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 and 64 points and the prefill")
     ap.add_argument("--no-workloads", action="store_true", help="skip the Qwen3-0.6B and Qwen3-32B workloads")
-    ap.add_argument("--design", choices=["vebonex", "tikizen", "sefalorn", "ruzunex"],
+    ap.add_argument("--design", choices=["vebonex", "tikizen", "sefalorn", "ruzunex", "dasusun"],
                     help="another workload: this design beside the closest model")
     ap.add_argument("--design-layers", type=int, default=8, help="layers of both models of --design")
     ap.add_argument("--design-steps", type=int, default=64, help="timed decode steps of --design")

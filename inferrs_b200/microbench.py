@@ -343,9 +343,11 @@ def joint(args) -> dict:
 
 def latent(args) -> dict:
     """The attention over cached latents alone: one prompt of ``tokens`` rows after ``context_before`` cached ones, or
-    ``batch`` single tokens over ``context`` latents each.  Flops: scores and sums over the latents, 4 R per head,
-    row and visible key; bytes: every visible latent once per request, queries and results."""
+    ``batch`` single tokens over ``context`` latents each, with ``rot`` more numbers per cached vector that join the
+    scores and a ``window`` (0: none).  Flops: scores and sums, 2 (R + rot) + 2 R per head, row and visible key; bytes:
+    every visible cached vector once per request, queries and results."""
     h, r, ps = args.heads, args.rank, args.page_size
+    rot_dim, window = getattr(args, "rot", 0), getattr(args, "window", 0) or None
     dev = torch.device("cuda")
     dtype = torch.float32 if args.dtype == "f32" else torch.bfloat16
     if args.form == "decode":
@@ -364,23 +366,113 @@ def latent(args) -> dict:
     row_request = torch.tensor([i for i, t in enumerate(new) for _ in range(t)], dtype=torch.int32, device=dev)
     n = sum(new)
     q = torch.randn(h, n, r, device=dev).to(dtype)
-    plane = torch.randn(n_pages, ps, r, device=dev).to(dtype)
+    q_rot, rot = None, None
+    if rot_dim:
+        q_rot = torch.randn(n, h, 128 + rot_dim, device=dev).to(dtype)[:, :, 128:]
+        cos, sin = (torch.randn(max(lens), rot_dim // 2, device=dev) for _ in range(2))
+        rot = kernels.LatentRotation(at=r, src=rot_dim, width=(rot_dim + 15) // 16 * 16, half=rot_dim // 2, cos=cos, sin=sin)
+    plane = torch.randn(n_pages, ps, r + (rot.width if rot else 0), device=dev).to(dtype)
     out = torch.empty(h, n, r, dtype=dtype, device=dev)
-    slices = args.slices or kernels.latent_slices(n, h, max(lens))
+    keys = max(lens) if window is None else min(max(lens), window + kernels.LATENT_TILE_KEYS)
+    slices = args.slices or kernels.latent_slices(n, h, keys)
     table = table.to(dev)
     tiles = None
     if args.form == "prefill" and slices == 1:     # as the engine runs prompt portions: two tokens of the request per block
         tt = kernels.LATENT_TILE_TOKENS
         row0 = torch.arange(0, n, tt, dtype=torch.int32, device=dev)
         tiles = (torch.zeros_like(row0), row0, row0.shape[0], torch.tensor([0, n], dtype=torch.int32, device=dev))
-    fn = lambda: kernels.latent_attention(q, plane, table, row_request, positions, r ** -0.5, None, out, slices, tiles)  # noqa: E731
+    fn = lambda: kernels.latent_attention(q, plane, table, row_request, positions, r ** -0.5, window, out, slices, tiles,  # noqa: E731
+                                          q_rot=q_rot, rot=rot)
     us = _time(fn, args.iters)
     el = 4 if dtype == torch.float32 else 2
-    pairs = sum(t * (c - t) + t * (t + 1) // 2 for c, t in zip(lens, new))
-    byts = el * (sum(lens) * r + 2 * n * h * r)
-    flops = 4 * h * r * pairs
-    return {"kernel": f"latent_attention/{args.form}", "heads": h, "rank": r, "rows": n, "keys": lens[0],
-            "slices": slices, "us": round(us, 2), "GBps": round(byts / us / 1e3, 1), "TFLOPs": round(flops / us / 1e6, 2)}
+    seen = lambda p: p + 1 if window is None else min(p + 1, window)          # noqa: E731
+    pairs = sum(seen(p) for c, t in zip(lens, new) for p in range(c - t, c))
+    touched = sum(c if window is None else min(c, window + t - 1) for c, t in zip(lens, new))
+    byts = el * (touched * (r + rot_dim) + n * h * (2 * r + rot_dim))
+    flops = (4 * r + 2 * rot_dim) * h * pairs
+    return {"kernel": f"latent_attention/{args.form}", "heads": h, "rank": r, "rot": rot_dim, "window": window, "rows": n,
+            "keys": lens[0], "slices": slices, "us": round(us, 2), "GBps": round(byts / us / 1e3, 1),
+            "TFLOPs": round(flops / us / 1e6, 2)}
+
+
+def latent_store(args) -> dict:
+    """The norms of both latents and the store into the pages, with ``rot`` numbers behind the latent that are turned
+    by position (0: none), for ``tokens`` rows of one request.  Bytes: the projection's columns, the query latent and the
+    cached vector."""
+    n, qr, r, rot_dim, ps = args.tokens, args.q_rank, args.rank, args.rot, 16
+    dev, dtype = torch.device("cuda"), torch.bfloat16
+    proj = torch.randn(n, qr + r + rot_dim, device=dev).to(dtype)
+    qw, kw = torch.randn(qr, device=dev).to(dtype), torch.randn(r, device=dev).to(dtype)
+    rot = None
+    if rot_dim:
+        cos, sin = (torch.randn(n, rot_dim // 2, device=dev) for _ in range(2))
+        rot = kernels.LatentRotation(at=r, src=rot_dim, width=(rot_dim + 15) // 16 * 16, half=rot_dim // 2, cos=cos, sin=sin)
+    n_pages = (n + ps - 1) // ps
+    plane = torch.zeros(n_pages, ps, r + (rot.width if rot else 0), dtype=dtype, device=dev)
+    table = torch.randperm(n_pages).to(torch.int32).to(dev)[None, :].contiguous()
+    cq = torch.empty(n, qr, dtype=dtype, device=dev)
+    zero, pos = torch.zeros(n, dtype=torch.int32, device=dev), torch.arange(n, dtype=torch.int32, device=dev)
+    us = _time(lambda: kernels.latent_norm_store(proj, 0, qw, cq, qr, kw, plane, table, zero, pos, 1e-5, rot=rot), args.iters)
+    byts = 2 * n * 2 * (qr + r + rot_dim)
+    return {"kernel": "latent_norm_store", "rows": n, "q_rank": qr, "rank": r, "rot": rot_dim, "us": round(us, 2),
+            "GBps": round(byts / us / 1e3, 1), "TFLOPs": 0.0}
+
+
+def residual(args) -> dict:
+    """What stands between two sub-layers, for ``tokens`` rows of ``width``.  impl ``sandwich``: the norm and scale on the
+    output, the addition, an average over ``planes`` earlier results (0: none), the next norm, and with ``taps`` > 0 (single
+    rows) the convolution; ``streams``: the update, read and norm of two streams in four parts; ``add``: addition and norm.
+    Bytes: every float32 and bfloat16 row once each way."""
+    n, w, planes = args.tokens, args.width, args.planes
+    dev, dtype = torch.device("cuda"), torch.bfloat16
+    y, out, weight = torch.randn(n, w, device=dev).to(dtype), torch.empty(n, w, dtype=dtype, device=dev), torch.randn(w, device=dev)
+    if args.impl == "streams":
+        x = torch.randn(n, 2, w, device=dev)
+        mix, gain, read = torch.eye(2, device=dev), torch.ones(2, device=dev), torch.ones(2, device=dev)
+        fn = lambda: kernels.stream_add_norm(x, y, mix, gain, read, weight, 4, 1e-5, out)           # noqa: E731
+        byts = n * w * (2 * 8 + 4)
+    elif args.impl == "add":
+        x = torch.randn(n, w, device=dev)
+        fn = lambda: kernels.add_rms_norm(x, y, weight, 1e-5, out)                                   # noqa: E731
+        byts = n * w * (8 + 4)
+    else:
+        x, post = torch.randn(n, w, device=dev), torch.randn(w, device=dev)
+        past = torch.randn(planes, n, w, device=dev) if planes else None
+        mix = torch.randn(planes + 1, device=dev) * 0.1 if planes else None
+        res = torch.empty(n, w, device=dev) if planes else None
+        conv = None
+        if args.taps:
+            state = torch.zeros(n, max(args.taps - 1, 1) * w, device=dev)
+            ids = torch.arange(n, dtype=torch.int32, device=dev)
+            conv = (torch.randn(args.taps, w, device=dev), state, 0, ids, ids)
+        fn = lambda: kernels.sandwich_norm(x, y, post, 1e-5, weight, 1e-5, out, residual=x, planes=past, mix=mix,   # noqa: E731
+                                           result=res, conv=conv)
+        byts = n * w * (8 + 4 + (planes + 1) * 4 * bool(planes) + 8 * max(args.taps - 1, 0))
+    us = _time(fn, args.iters)
+    return {"kernel": f"residual/{args.impl}", "rows": n, "width": w, "planes": planes, "taps": args.taps, "us": round(us, 2),
+            "GBps": round(byts / us / 1e3, 1), "TFLOPs": 0.0}
+
+
+def activation(args) -> dict:
+    """What stands between the two products of a feed-forward without a gate, for ``tokens`` rows of ``inner``: ``gelu``, the
+    ``poly`` activation of unit-rms terms, or (``product``) the up product of ``k`` inputs whose read-back takes gelu and
+    (``plain-product``) the same without."""
+    n, f, k = args.tokens, args.inner, args.k
+    dev, dtype = torch.device("cuda"), torch.bfloat16
+    z, out = torch.randn(n, f, device=dev).to(dtype), torch.empty(n, f, dtype=dtype, device=dev)
+    byts, flops = 4 * n * f, 0
+    if args.impl == "gelu":
+        fn = lambda: kernels.gelu_rows(z, out)                                                       # noqa: E731
+    elif args.impl == "poly":
+        coef = torch.tensor([0.5, 0.3, 0.2, 0.0], device=dev)
+        fn = lambda: kernels.poly_norm(z, coef, 1e-5, out)                                           # noqa: E731
+    else:
+        x, w = torch.randn(n, k, device=dev).to(dtype), (torch.randn(f, k, device=dev) * 0.02).to(dtype)
+        fn = lambda: kernels.gemm_tn_tcgen05(x, w, out, gelu=args.impl == "product")                 # noqa: E731
+        byts, flops = 2 * (f * k + n * k + n * f), 2 * n * f * k
+    us = _time(fn, args.iters)
+    return {"kernel": f"activation/{args.impl}", "rows": n, "inner": f, "us": round(us, 2), "GBps": round(byts / us / 1e3, 1),
+            "TFLOPs": round(flops / us / 1e6, 2)}
 
 
 def chain(args) -> dict:
@@ -757,9 +849,36 @@ def main(argv=None) -> int:
     la.add_argument("--heads", type=int, default=16)
     la.add_argument("--rank", type=int, default=512)
     la.add_argument("--slices", type=int, default=0, help="slices of a row's keys (0: as the engine chooses)")
+    la.add_argument("--rot", type=int, default=0, help="numbers of a cached vector behind the latent, for the scores alone")
+    la.add_argument("--window", type=int, default=0)
     la.add_argument("--page-size", type=int, default=16)
     la.add_argument("--iters", type=int, default=20)
     la.set_defaults(fn=latent)
+
+    ls = sub.add_parser("latent-store")
+    ls.add_argument("--tokens", type=int, default=2048)
+    ls.add_argument("--q-rank", type=int, default=768)
+    ls.add_argument("--rank", type=int, default=512)
+    ls.add_argument("--rot", type=int, default=64)
+    ls.add_argument("--iters", type=int, default=20)
+    ls.set_defaults(fn=latent_store)
+
+    rs = sub.add_parser("residual")
+    rs.add_argument("--impl", choices=["sandwich", "streams", "add"], default="sandwich")
+    rs.add_argument("--tokens", type=int, default=2048)
+    rs.add_argument("--width", type=int, default=2048)
+    rs.add_argument("--planes", type=int, default=0)
+    rs.add_argument("--taps", type=int, default=0)
+    rs.add_argument("--iters", type=int, default=20)
+    rs.set_defaults(fn=residual)
+
+    ac = sub.add_parser("activation")
+    ac.add_argument("--impl", choices=["gelu", "poly", "product", "plain-product"], default="gelu")
+    ac.add_argument("--tokens", type=int, default=2048)
+    ac.add_argument("--inner", type=int, default=8192)
+    ac.add_argument("--k", type=int, default=2048)
+    ac.add_argument("--iters", type=int, default=20)
+    ac.set_defaults(fn=activation)
     c = sub.add_parser("chain")
     c.add_argument("--impl", choices=["library", "tcgen05", "folded", "persistent"], default="library",
                    help="folded: the products with the norms folded in, one kernel each; persistent: the same four as one kernel")
