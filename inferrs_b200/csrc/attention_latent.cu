@@ -241,6 +241,10 @@ __device__ __forceinline__ void lm_cp_async16(void* dst, const void* src, int sr
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" :: "r"(d), "l"(src), "r"(src_bytes) : "memory");
 }
 
+// Vectors of a multiple of 64 numbers lie in shared memory without padding: at 512 + 64 numbers two blocks then just fit
+// on an SM (228 KB with the 1 KB that each block costs).
+__host__ __device__ constexpr int lm_swizzle(int rk) { return rk % 64 == 0 ? 7 : 0; }
+
 // NT: n-tiles of 8 columns per warp in the second product, R = 32 * NT.  TT: tokens per block.  TT = 1: a block per
 // row (blockIdx.x), any slices.  TT = 2: a block per tile of up to two tokens of one request, named by a tile list
 // (tile_req[i] < 0: no tile); the two tokens' queries meet every tile of latents together, so a prompt's latents
@@ -255,9 +259,13 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
                             const int* __restrict__ tile_row0, const int* __restrict__ q_start, int n_heads, float scale,
                             int window, int n_slices, __nv_bfloat16* __restrict__ out, long o_row, long o_head,
                             float* __restrict__ ws_acc, float* __restrict__ ws_ml, const LatentRot rot) {
-    constexpr int R = 32 * NT, LDP = LM_KEYS + LM_PAD, MR = TT * LM_ROWS;
+    constexpr int R = 32 * NT, MR = TT * LM_ROWS;
     const int RK = ROT ? R + rot.width : R;              // numbers of a cached vector
-    const int LDC = RK + LM_PAD;
+    const int sw = ROT ? lm_swizzle(RK) : 0;             // rows without padding, their 16-byte places exchanged
+    const int LDC = RK + (sw ? 0 : LM_PAD), LDP = LM_KEYS + (sw ? 0 : LM_PAD);
+    // element `col` (a multiple of eight) of row r: the place's low three bits are turned over by the row's, so that
+    // eight rows' equal columns lie in eight different groups of banks
+    auto at = [sw](int r, int ld, int col) { return r * ld + (((col >> 3) ^ (r & sw)) << 3); };
     extern __shared__ __align__(16) unsigned char lm_smem[];
     __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(lm_smem);          // [TT * 16][LDC]
     __nv_bfloat16* c_s = q_s + MR * LDC;                                     // [64][LDC]
@@ -292,14 +300,14 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
         const int tok = m / LM_ROWS, h = head0 + m % LM_ROWS;
         const bool ok = h < n_heads && tok < n_tok;
         const __nv_bfloat16* src = q + (long)(row + (ok ? tok : 0)) * q_row + (long)min(h, n_heads - 1) * q_head + ch * 8;
-        lm_cp_async16(q_s + m * LDC + ch * 8, src, ok ? 16 : 0);
+        lm_cp_async16(q_s + at(m, LDC, ch * 8), src, ok ? 16 : 0);
     }
     if constexpr (ROT) {                              // their rotated parts, turned as they are fetched
         for (int i = threadIdx.x; i < MR * rot.width; i += blockDim.x) {
             const int m = i / rot.width, e = i % rot.width;
             const int tok = m / LM_ROWS, h = head0 + m % LM_ROWS;
             const bool ok = h < n_heads && tok < n_tok;
-            q_s[m * LDC + R + e] = __float2bfloat16_rn(ok ? latent_rot_value<__nv_bfloat16>(rot, row + tok, h, e, pos0 + tok) : 0.0f);
+            q_s[at(m, LDC, (R + e) & ~7) + (e & 7)] = __float2bfloat16_rn(ok ? latent_rot_value<__nv_bfloat16>(rot, row + tok, h, e, pos0 + tok) : 0.0f);
         }
     }
     // two threads per key: the page is looked up once per key and tile, each thread copies half of the latent
@@ -315,11 +323,10 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
                 bytes = 16;
             }
         }
-        __nv_bfloat16* dst = c_s + jj * LDC;
 #pragma unroll
-        for (int ch = half; ch < R / 8; ch += 2) lm_cp_async16(dst + ch * 8, bytes ? src + ch * 8 : src, bytes);
+        for (int ch = half; ch < R / 8; ch += 2) lm_cp_async16(c_s + at(jj, LDC, ch * 8), bytes ? src + ch * 8 : src, bytes);
         if constexpr (ROT)
-            for (int ch = R / 8 + half; ch < RK / 8; ch += 2) lm_cp_async16(dst + ch * 8, bytes ? src + ch * 8 : src, bytes);
+            for (int ch = R / 8 + half; ch < RK / 8; ch += 2) lm_cp_async16(c_s + at(jj, LDC, ch * 8), bytes ? src + ch * 8 : src, bytes);
     };
     if (t0 < t1) load_tile(t0);
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -351,11 +358,11 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
             }
         auto score_step = [&](int ks, bool second) {
             uint32_t b0, b1, b2, b3;
-            lm_ldmatrix_x4(b0, b1, b2, b3, ct + (warp * 16 + (lane & 7) + (lane >> 4) * 8) * LDC + ks * 16 + ((lane >> 3) & 1) * 8);
+            lm_ldmatrix_x4(b0, b1, b2, b3, ct + at(warp * 16 + (lane & 7) + (lane >> 4) * 8, LDC, ks * 16 + ((lane >> 3) & 1) * 8));
 #pragma unroll
             for (int tk = 0; tk < TT; ++tk) {
                 uint32_t a0, a1, a2, a3;
-                lm_ldmatrix_x4(a0, a1, a2, a3, q_s + (tk * LM_ROWS + (lane & 15)) * LDC + ks * 16 + (lane >> 4) * 8);
+                lm_ldmatrix_x4(a0, a1, a2, a3, q_s + at(tk * LM_ROWS + (lane & 15), LDC, ks * 16 + (lane >> 4) * 8));
                 if (second) {
                     lm_mma(sd[tk][0], a0, a1, a2, a3, b0, b1);
                     lm_mma(sd[tk][1], a0, a1, a2, a3, b2, b3);
@@ -416,9 +423,9 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
                     p[c] = (sc[tk][i][c] == -INFINITY) ? 0.0f : expf(sc[tk][i][c] - m_new[c >> 1]);
                     sm[c >> 1] += p[c];
                 }
-                const int col = warp * 16 + i * 8 + 2 * (lane & 3);
-                *reinterpret_cast<__nv_bfloat162*>(p_s + (tk * LM_ROWS + r_lo) * LDP + col) = __floats2bfloat162_rn(p[0], p[1]);
-                *reinterpret_cast<__nv_bfloat162*>(p_s + (tk * LM_ROWS + r_hi) * LDP + col) = __floats2bfloat162_rn(p[2], p[3]);
+                const int col = warp * 16 + i * 8, in8 = 2 * (lane & 3);
+                *reinterpret_cast<__nv_bfloat162*>(p_s + at(tk * LM_ROWS + r_lo, LDP, col) + in8) = __floats2bfloat162_rn(p[0], p[1]);
+                *reinterpret_cast<__nv_bfloat162*>(p_s + at(tk * LM_ROWS + r_hi, LDP, col) + in8) = __floats2bfloat162_rn(p[2], p[3]);
             }
 #pragma unroll
             for (int k = 0; k < 2; ++k) {
@@ -450,11 +457,11 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long q_row, lon
             uint32_t a[TT][4];
 #pragma unroll
             for (int tk = 0; tk < TT; ++tk)
-                lm_ldmatrix_x4(a[tk][0], a[tk][1], a[tk][2], a[tk][3], p_s + (tk * LM_ROWS + (lane & 15)) * LDP + kk * 16 + (lane >> 4) * 8);
+                lm_ldmatrix_x4(a[tk][0], a[tk][1], a[tk][2], a[tk][3], p_s + at(tk * LM_ROWS + (lane & 15), LDP, kk * 16 + (lane >> 4) * 8));
 #pragma unroll
             for (int i = 0; i < NT; i += 2) {
                 uint32_t b0, b1, b2, b3;
-                lm_ldmatrix_x4_trans(b0, b1, b2, b3, ct + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LDC + warp * (R / 4) + i * 8 + (lane >> 4) * 8);
+                lm_ldmatrix_x4_trans(b0, b1, b2, b3, ct + at(kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, LDC, warp * (R / 4) + i * 8 + (lane >> 4) * 8));
 #pragma unroll
                 for (int tk = 0; tk < TT; ++tk) {
                     lm_mma(o[tk][i], a[tk][0], a[tk][1], a[tk][2], a[tk][3], b0, b1);
@@ -508,13 +515,12 @@ static int launch_latent_mma(const void* q, long q_row, long q_head, const void*
                              const int* tile_req, const int* tile_row0, const int* q_start, int n_blocks, int n_heads,
                              float scale, int window, int n_slices, void* out, long o_row, long o_head, float* ws_acc,
                              float* ws_ml, const LatentRot& rot, cudaStream_t stream) {
-    constexpr int R = 32 * NT, LDP = LM_KEYS + LM_PAD, MR = TT * LM_ROWS;
-    auto smem_for = [](int width) {
-        const int ldc = R + width + LM_PAD;
-        return (size_t)(MR * ldc + LM_KEYS * ldc + MR * LDP) * 2 + 8 * MR * sizeof(float);
+    constexpr int R = 32 * NT, MR = TT * LM_ROWS;
+    auto smem_for = [](int width, int pad) {
+        return (size_t)((MR + LM_KEYS) * (R + width + pad) + MR * (LM_KEYS + pad)) * 2 + 8 * MR * sizeof(float);
     };
-    const size_t smem = smem_for(ROT ? rot.width : 0);
-    const size_t smem_most = smem_for(ROT ? LM_MOST_ROT : 0);     // the permission is given once per device, for the most
+    const size_t smem = ROT ? smem_for(rot.width, lm_swizzle(R + rot.width) ? 0 : LM_PAD) : smem_for(0, LM_PAD);
+    const size_t smem_most = smem_for(ROT ? LM_MOST_ROT : 0, LM_PAD);     // the permission is given once per device, for the most
     if (smem_most > 48 * 1024) {
         const int e = ib_allow_dynamic_smem(latent_mma_smem_set[ROT][TT - 1][NT], latent_attention_mma_kernel<NT, TT, ROT>,
                                             smem_most);
