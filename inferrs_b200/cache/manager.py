@@ -11,7 +11,8 @@ Here the cache is a list of *groups*.  A group is a set of caches (one per
 schedule entry that writes keys and values) with the same needs: the same
 number of key/value heads, head size and visibility (all keys, or a window).
 Each group has a page pool and a block table per request of its own; a window
-group gives pages back as soon as the window has passed them.  Beside the
+group gives pages back as soon as the window has passed them (but not the
+pages of a sequence's first tokens where these stay visible).  Beside the
 pages there are *state slots*: one slot per live request, the index into
 per-request tensors of fixed size (sampler state, and the state of mixers that
 keep one).
@@ -48,6 +49,7 @@ class GroupLayout:
 
     name: str
     window: Optional[int] = None  # None: all keys; w: a query at i sees keys j with i - w < j <= i
+    keep_first: int = 0           # beside its window a query also sees the sequence's first keys, j < keep_first
 
 
 _ERR_UNKNOWN_REQUEST, _ERR_ALREADY_LIVE, _ERR_NO_SLOT, _ERR_OUT_OF_PAGES = -1, -2, -3, -4
@@ -63,7 +65,7 @@ def host_library():
     if _LIB is None:
         lib = load_library("host_runtime")
         i, p, l = ctypes.c_int, ctypes.c_void_p, ctypes.c_int64
-        lib.ibh_cache_new.argtypes = [i, p, p, i, i]
+        lib.ibh_cache_new.argtypes = [i, p, p, p, i, i]
         lib.ibh_cache_new.restype = p
         lib.ibh_cache_delete.argtypes = [p]
         lib.ibh_cache_delete.restype = None
@@ -124,6 +126,8 @@ class CacheManager:
         for g in groups:
             if g.window is not None and g.window <= 0:
                 raise CacheError(f"group {g.name}: window must be positive, got {g.window}")
+            if g.keep_first < 0:
+                raise CacheError(f"group {g.name}: keep_first must not be negative, got {g.keep_first}")
         for n in n_pages:
             if n <= 0:
                 raise CacheError(f"a page pool needs at least one page, got {n}")
@@ -132,8 +136,9 @@ class CacheManager:
         self.max_requests = max_requests
         self._lib = host_library()
         windows = (ctypes.c_int * len(groups))(*[-1 if g.window is None else g.window for g in groups])
+        keeps = (ctypes.c_int * len(groups))(*[int(g.keep_first) for g in groups])
         counts = (ctypes.c_int * len(groups))(*[int(n) for n in n_pages])
-        self._h = self._lib.ibh_cache_new(len(groups), windows, counts, page_size, max_requests)
+        self._h = self._lib.ibh_cache_new(len(groups), windows, keeps, counts, page_size, max_requests)
         if not self._h:
             raise CacheError("the native cache manager refused these sizes")
         self.pools = [_PoolView(self, g, int(n)) for g, n in enumerate(n_pages)]

@@ -32,6 +32,8 @@ class KVNeed:
     # size of a value head where it differs from a key head's (None: the same; such a group keeps its values in
     # a tensor of their own)
     value_dim: Optional[int] = None
+    # how many of a sequence's first tokens stay visible beside the window
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
@@ -77,7 +79,7 @@ class CacheStorage:
         if any(k.planes not in (1, 2) for k in keys):
             raise ValueError("a cache has one plane (latents) or two (keys and values)")
         self.layouts = [GroupLayout(name=f"group{g}(heads={k.n_kv_heads},dim={k.head_dim},window={k.window})",
-                                    window=k.window) for g, k in enumerate(keys)]
+                                    window=k.window, keep_first=k.keep_first) for g, k in enumerate(keys)]
         self.n_pages = list(n_pages_per_group) if n_pages_per_group is not None else [n_pages] * len(keys)
         if any(k.value_dim is not None and k.planes != 2 for k in keys):
             raise ValueError("values of a size of their own need a cache of two planes")

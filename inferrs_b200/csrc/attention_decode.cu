@@ -64,8 +64,13 @@ struct Params {
     const int* reqs;           // [R] or null: its request (row of the block table); a negative row is no work
     int max_pages, page_size, n_pages, n_heads, n_kv_heads, window, max_splits, min_tiles;
     float scale_log2;
+    float cap_k, cap_c;        // see ib_capped_log2
+    IbScoreOptions opt;
 };
 
+// OPTIONS: a factor, a slope and a sink per head, a cap on the scores, a sequence's first keys beside the window, a
+// gate per head.
+template <bool OPTIONS>
 __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constant__ CUtensorMap map_k,
                                                             const __grid_constant__ CUtensorMap map_v, const Params P) {
     extern __shared__ unsigned char raw_smem[];
@@ -95,15 +100,17 @@ __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constan
     const int G = P.n_heads / P.n_kv_heads;
     const int pos = P.positions[row];
     const int lo = ib_first_visible(pos, P.window);
-    const int t_first = lo / KEYS, t_last = pos / KEYS + 1;
-    const int n_all = t_last - t_first;
+    // the request's tiles: those that hold kept keys, then the window's from t_first on
+    const int keep = OPTIONS ? P.opt.keep_first : 0;
+    const int t_first = lo / KEYS, n_kept = ib_kept_tiles(keep, t_first, KEYS);
+    const int n_all = n_kept + pos / KEYS + 1 - t_first;
     int n_splits = (n_all + P.min_tiles - 1) / P.min_tiles;
     if (n_splits > P.max_splits) n_splits = P.max_splits;
     if (split >= n_splits) { asm volatile("griddepcontrol.wait;" ::: "memory"); return; }   // an unused slice
     const int per = (n_all + n_splits - 1) / n_splits;
-    const int t_begin = t_first + split * per;
-    const int t_end = t_begin + per < t_last ? t_begin + per : t_last;
-    const int n_tiles = t_end > t_begin ? t_end - t_begin : 0;
+    const int i_begin = split * per;                          // this slice's tiles: places i_begin .. of that list
+    const int i_end = i_begin + per < n_all ? i_begin + per : n_all;
+    const int n_tiles = i_end > i_begin ? i_end - i_begin : 0;
 
     if (threadIdx.x == 0) {
         for (int s = 0; s < STAGES; ++s) { mbar_init(full0 + 8 * s, 1); mbar_init(empty0 + 8 * s, 4); }
@@ -133,7 +140,7 @@ __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constan
         const int pages_per_tile = KEYS / P.page_size;
         auto lookup = [&](int i) -> int {
             if (lane >= pages_per_tile) return 0;
-            const int j = (t_begin + i) * KEYS + lane * P.page_size;
+            const int j = ib_nth_tile(i_begin + i, n_kept, t_first) * KEYS + lane * P.page_size;
             int page = (j <= pos && j / P.page_size < P.max_pages) ? bt[j / P.page_size] : -1;
             // No page (beyond the request, or given back): the copy is aimed past the last page, where TMA reads
             // nothing and fills the tile with zeros.  No query sees these keys, but their values are multiplied
@@ -144,7 +151,7 @@ __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constan
         int page_next = n_tiles > 0 ? lookup(0) : 0;
         // tiles that end before this step's position hold only keys of earlier steps: up to a ring of them
         // is asked for before the kernels before this one are waited for
-        int n_early = pos / KEYS - t_begin;
+        int n_early = n_all - 1 - i_begin;      // the list's last tile is the one that holds this step's position
         n_early = n_early < 0 ? 0 : (n_early > n_tiles ? n_tiles : n_early);
         n_early = n_early > STAGES ? STAGES : n_early;
         bool waited = false;
@@ -182,6 +189,16 @@ __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constan
             ldmatrix_x4(qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], smem_u32(sq + r * D + c * 8));
         }
         const bool row_ok[2] = {gid < G, gid + 8 < G};
+        float scale_r[2] = {P.scale_log2, P.scale_log2}, slope_r[2] = {0.0f, 0.0f};
+        if (OPTIONS) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                if (!row_ok[h]) continue;
+                const int head = kvh * G + gid + 8 * h;
+                if (P.opt.head_scale) scale_r[h] *= P.opt.head_scale[head];
+                if (P.opt.slopes) slope_r[h] = P.opt.slopes[head] * 1.4426950408889634f;
+            }
+        }
         for (int i = 0; i < n_tiles; ++i) {
             const int s = i % STAGES;
             if (ok && !mbar_wait(full0 + 8 * s, (i / STAGES) & 1, 2)) ok = false;
@@ -201,15 +218,21 @@ __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constan
                 mma16816(sc[0], qf[ks], b0, b1);
                 mma16816(sc[1], qf[ks], b2, b3);
             }
+            const int tile_key = ib_nth_tile(i_begin + i, n_kept, t_first) * KEYS;
             float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
             for (int n = 0; n < 2; ++n)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int h = e >> 1;
-                    const int j = (t_begin + i) * KEYS + key0 + n * 8 + 2 * tig + (e & 1);
-                    const bool vis = row_ok[h] && j >= lo && j <= pos;
-                    sc[n][e] = vis ? sc[n][e] * P.scale_log2 : -INFINITY;
+                    const int j = tile_key + key0 + n * 8 + 2 * tig + (e & 1);
+                    const bool vis = row_ok[h] && ib_visible(j, lo, pos, keep);
+                    float x = sc[n][e] * scale_r[h];
+                    if (OPTIONS) {
+                        x -= slope_r[h] * (float)(pos - j);
+                        if (P.opt.cap > 0.0f) x = ib_capped_log2(x, P.cap_k, P.cap_c);
+                    }
+                    sc[n][e] = vis ? x : -INFINITY;
                     mx[h] = fmaxf(mx[h], sc[n][e]);
                 }
             float corr[2], msafe[2];
@@ -278,7 +301,35 @@ __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constan
         }
     }
     __syncthreads();
-    const long head0 = (long)row * P.n_heads + kvh * G;       // of q and out
+    __nv_bfloat16* const out_row = P.out + row * P.opt.out_ld;
+    // a row's end: the sink joins the row's sum L (M its maximum), then the gate; returns the factor on the output
+    auto finish = [&](int g, float M, float L) -> float {
+        const int head = kvh * G + g;
+        float f = 1.0f;
+        if (P.opt.sinks) {
+            const float sink = P.opt.sinks[head] * 1.4426950408889634f;
+            const float m_new = fmaxf(M, sink);
+            f = M == -INFINITY ? 0.0f : exp2f(M - m_new);
+            L = L * f + exp2f(sink - m_new);
+        }
+        return L > 0.0f ? f / L * ib_head_gate(P.opt, row, head) : 0.0f;
+    };
+    auto store4 = [&](int g, int e, float4 acc, float M, float L) {
+        __nv_bfloat162 lo2, hi2;
+        if (OPTIONS) {
+            const float f = finish(g, M, L);
+            lo2 = __floats2bfloat162_rn(acc.x * f, acc.y * f);
+            hi2 = __floats2bfloat162_rn(acc.z * f, acc.w * f);
+        } else {
+            if (!(L > 0.0f)) { acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f); L = 1.0f; }
+            lo2 = __floats2bfloat162_rn(acc.x / L, acc.y / L);
+            hi2 = __floats2bfloat162_rn(acc.z / L, acc.w / L);
+        }
+        uint2 w;
+        w.x = *reinterpret_cast<unsigned*>(&lo2);
+        w.y = *reinterpret_cast<unsigned*>(&hi2);
+        *reinterpret_cast<uint2*>(out_row + (kvh * G + g) * D + e) = w;
+    };
     const long part0 = (long)place * P.n_heads + kvh * G;     // of the slices' scratch
     for (int idx = threadIdx.x; idx < G * (D / 4); idx += THREADS) {   // four elements per thread: one pass
         const int g = idx / (D / 4), e = (idx - g * (D / 4)) * 4;
@@ -303,13 +354,7 @@ __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constan
                 P.part_ml[((part0 + g) * P.max_splits + split) * 2 + 1] = L;
             }
         } else {
-            if (!(L > 0.0f)) { acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f); L = 1.0f; }
-            __nv_bfloat162 lo2 = __floats2bfloat162_rn(acc.x / L, acc.y / L);
-            __nv_bfloat162 hi2 = __floats2bfloat162_rn(acc.z / L, acc.w / L);
-            uint2 w2;
-            w2.x = *reinterpret_cast<unsigned*>(&lo2);
-            w2.y = *reinterpret_cast<unsigned*>(&hi2);
-            *reinterpret_cast<uint2*>(P.out + (head0 + g) * D + e) = w2;
+            store4(g, e, acc, M, L);
         }
     }
     if (n_splits > 1) {
@@ -354,13 +399,7 @@ __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constan
                         }
                     }
                 }
-                if (!(L > 0.0f)) { acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f); L = 1.0f; }
-                __nv_bfloat162 lo2 = __floats2bfloat162_rn(acc.x / L, acc.y / L);
-                __nv_bfloat162 hi2 = __floats2bfloat162_rn(acc.z / L, acc.w / L);
-                uint2 w;
-                w.x = *reinterpret_cast<unsigned*>(&lo2);
-                w.y = *reinterpret_cast<unsigned*>(&hi2);
-                *reinterpret_cast<uint2*>(P.out + (head0 + g) * D + e) = w;
+                store4(g, e, acc, M, L);
             }
         }
     }
@@ -380,7 +419,9 @@ IB_EXPORT int ib_paged_attention_decode(const void* q, const void* k_pages, cons
                                         int max_pages, int page_size, int n_pages, const int* positions, int n_rows,
                                         int n_heads, int n_kv_heads, int head_dim, float scale, int window, void* out,
                                         int max_splits, int min_tiles, float* part_o, float* part_ml, int* counters,
-                                        const int* rows, const int* reqs, cudaStream_t stream) {
+                                        const int* rows, const int* reqs, const float* head_scale, const float* slopes,
+                                        const float* sinks, float cap, int keep_first, const void* gate, long gate_ld,
+                                        long out_ld, cudaStream_t stream) {
     if (n_rows <= 0) return IB_OK;
     if (min_tiles <= 0) return IB_ERR_ARGUMENT;
     if ((rows == nullptr) != (reqs == nullptr)) return IB_ERR_ARGUMENT;
@@ -389,6 +430,9 @@ IB_EXPORT int ib_paged_attention_decode(const void* q, const void* k_pages, cons
     const int G = n_heads / n_kv_heads;
     if (head_dim != dec::D || dec::KEYS % page_size || page_size < 8 || G > 16) return IB_ERR_UNSUPPORTED;
     if (max_splits > 1 && (part_o == nullptr || part_ml == nullptr || counters == nullptr)) return IB_ERR_ARGUMENT;
+    if (keep_first < 0 || out_ld < (long)n_heads * head_dim || out_ld % 4 || ((uintptr_t)out & 7) ||
+        (gate != nullptr && gate_ld < n_heads))
+        return IB_ERR_ARGUMENT;
     dec::EncodeTiled enc = dec::encode_fn();
     if (enc == nullptr) return IB_ERR_UNSUPPORTED;
     CUtensorMap mk, mv;
@@ -409,10 +453,19 @@ IB_EXPORT int ib_paged_attention_decode(const void* q, const void* k_pages, cons
     P.n_pages = n_pages; P.n_heads = n_heads; P.n_kv_heads = n_kv_heads; P.window = window; P.max_splits = max_splits;
     P.min_tiles = min_tiles;
     P.scale_log2 = scale * 1.4426950408889634f;
+    P.cap_k = cap > 0.0f ? 2.0f / cap : 0.0f;      // the scores carry the factor log2(e) already
+    P.cap_c = cap * 1.4426950408889634f;
+    P.opt = {head_scale, slopes, sinks, cap, keep_first, (const act_t*)gate, gate_ld, out_ld};
     const size_t smem = 2 * dec::STAGES * dec::TILE_BYTES + 16 * dec::D * 2 + (2 * dec::STAGES + 1) * 8 + 1024;
-    static IbDeviceSet configured;   // the attribute is kept per device
-    if (const int e = ib_allow_dynamic_smem(configured, dec::decode_kernel, smem)) return e;
-    ib_launch(dec::decode_kernel, dim3(n_rows, n_kv_heads, max_splits), dec::THREADS, smem, stream, mk, mv, P);
+    static IbDeviceSet configured, configured_options;   // the attribute is kept per device
+    const dim3 grid(n_rows, n_kv_heads, max_splits);
+    if (head_scale != nullptr || slopes != nullptr || sinks != nullptr || cap > 0.0f || gate != nullptr || keep_first > 0) {
+        if (const int e = ib_allow_dynamic_smem(configured_options, dec::decode_kernel<true>, smem)) return e;
+        ib_launch(dec::decode_kernel<true>, grid, dec::THREADS, smem, stream, mk, mv, P);
+    } else {
+        if (const int e = ib_allow_dynamic_smem(configured, dec::decode_kernel<false>, smem)) return e;
+        ib_launch(dec::decode_kernel<false>, grid, dec::THREADS, smem, stream, mk, mv, P);
+    }
     return ib_launch_status();
 }
 
@@ -436,7 +489,8 @@ IB_EXPORT int ib_attention_decode_error_async(int* out, cudaStream_t stream) {
 
 IB_EXPORT int ib_paged_attention_decode(const void*, const void*, const void*, const int*, int, int, int, const int*, int,
                                         int, int, int, float, int, void*, int, int, float*, float*, int*, const int*,
-                                        const int*, cudaStream_t) {
+                                        const int*, const float*, const float*, const float*, float, int, const void*, long,
+                                        long, cudaStream_t) {
     return IB_ERR_UNSUPPORTED;
 }
 

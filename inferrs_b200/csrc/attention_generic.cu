@@ -21,7 +21,8 @@
 // Three more options, each a number per head (absent: not applied).  head_scale[h] multiplies head h's scaled score
 // (a learned temperature).  slopes[h] * (pos - j) is taken off the score (a bias that grows linearly with the
 // distance).  sinks[h]: every row's softmax gets one more term, exp(sinks[h]), in its denominator only; no key or
-// value belongs to it, and neither the scale nor the factor nor the slope touches it.
+// value belongs to it, and neither the scale nor the factor nor the slope touches it.  The other options (a cap on the
+// scores, a sequence's first keys beside the window, a gate per head) are those of IbScoreOptions.
 #include "common.cuh"
 
 #define ATT_WARPS 4
@@ -32,8 +33,7 @@ __global__ void paged_attention_generic_kernel(
     const int* __restrict__ block_table, int max_pages, int page_size, int n_pages,
     const int* __restrict__ row_request, const int* __restrict__ positions, int n_heads, int n_kv_heads,
     int head_dim, int v_dim, float scale, int window, act_t* __restrict__ out,
-    const float* __restrict__ dist_bias, int bias_len, const float* __restrict__ head_scale,
-    const float* __restrict__ slopes, const float* __restrict__ sinks) {
+    const float* __restrict__ dist_bias, int bias_len, const IbScoreOptions opt) {
     extern __shared__ float smem[];
     ib_grid_dependency_sync();
     const int row = blockIdx.x;
@@ -52,8 +52,8 @@ __global__ void paged_attention_generic_kernel(
     const act_t* qr = q + ((long)row * n_heads + head) * dq;
     for (int e = lane; e < dq; e += 32) qs[e] = ib_to_float(qr[e]);
     const float* bias_h = dist_bias ? dist_bias + (long)head * bias_len : nullptr;
-    const float scale_h = head_scale ? scale * head_scale[head] : scale;
-    const float slope_h = slopes ? slopes[head] : 0.0f;
+    const float scale_h = opt.head_scale ? scale * opt.head_scale[head] : scale;
+    const float slope_h = opt.slopes ? opt.slopes[head] : 0.0f;
     __syncwarp();
 
     float acc[DPL];
@@ -61,9 +61,12 @@ __global__ void paged_attention_generic_kernel(
     for (int k = 0; k < DPL; ++k) acc[k] = 0.0f;
     float m = -INFINITY, l = 0.0f;
 
-    for (int j0 = (lo / 32) * 32; j0 <= pos; j0 += 32) {
+    const int n_kept = ib_kept_tiles(opt.keep_first, lo / 32, 32);
+    for (int i = 0; ; ++i) {
+        const int j0 = ib_nth_tile(i, n_kept, lo / 32) * 32;
+        if (j0 > pos) break;
         const int j = j0 + lane;
-        const bool valid = j >= lo && j <= pos;
+        const bool valid = ib_visible(j, lo, pos, opt.keep_first);
         float s = -INFINITY;
         long off = 0;      // the key's place counted in heads' rows; times d its key, times v_dim its value
         if (valid) {
@@ -83,6 +86,7 @@ __global__ void paged_attention_generic_kernel(
                 }
                 s = dot * scale_h - slope_h * (float)(pos - j);
                 if (bias_h) s -= bias_h[pos - j < bias_len ? pos - j : bias_len - 1];
+                if (opt.cap > 0.0f) s = opt.cap * tanhf(s / opt.cap);
             }
         }
         const float m_new = fmaxf(m, ib_warp_max(s));
@@ -105,16 +109,16 @@ __global__ void paged_attention_generic_kernel(
         }
         m = m_new;
     }
-    if (sinks) {        // the place without a key: it adds to the denominator and to nothing else
-        const float sink = sinks[head];
+    if (opt.sinks) {        // the place without a key: it adds to the denominator and to nothing else
+        const float sink = opt.sinks[head];
         const float m_new = fmaxf(m, sink);
         const float corr = (m == -INFINITY) ? 0.0f : expf(m - m_new);
         l = l * corr + expf(sink - m_new);
 #pragma unroll
         for (int k = 0; k < DPL; ++k) acc[k] *= corr;
     }
-    const float inv = l > 0.0f ? 1.0f / l : 0.0f;
-    act_t* dst = out + ((long)row * n_heads + head) * v_dim;
+    const float inv = (l > 0.0f ? 1.0f / l : 0.0f) * ib_head_gate(opt, row, head);
+    act_t* dst = out + row * opt.out_ld + (long)head * v_dim;
 #pragma unroll
     for (int k = 0; k < DPL; ++k) {
         const int e = lane + 32 * k;
@@ -127,12 +131,15 @@ IB_EXPORT int ib_paged_attention_generic(const void* q, const void* k_pages, con
                                          const int* row_request, const int* positions, int n_rows, int n_heads,
                                          int n_kv_heads, int head_dim, int v_dim, float scale, int window, void* out,
                                          int joint, const float* dist_bias, int bias_len, const float* head_scale,
-                                         const float* slopes, const float* sinks, cudaStream_t stream) {
+                                         const float* slopes, const float* sinks, float cap, int keep_first,
+                                         const void* gate, long gate_ld, long out_ld, cudaStream_t stream) {
     if (n_rows <= 0) return IB_OK;
     if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads || head_dim <= 0 || page_size <= 0 || max_pages <= 0)
         return IB_ERR_ARGUMENT;
     if (v_dim <= 0) return IB_ERR_ARGUMENT;
     if (dist_bias != nullptr && bias_len <= 0) return IB_ERR_ARGUMENT;
+    if (keep_first < 0 || out_ld < (long)n_heads * v_dim || (gate != nullptr && gate_ld < n_heads)) return IB_ERR_ARGUMENT;
+    const IbScoreOptions opt = {head_scale, slopes, sinks, cap, keep_first, (const act_t*)gate, gate_ld, out_ld};
     const int dq = joint ? n_kv_heads * head_dim : head_dim;
     if (head_dim > 512 || v_dim > 512 || dq > 2048) return IB_ERR_UNSUPPORTED;
     const dim3 grid(n_rows, (n_heads + ATT_WARPS - 1) / ATT_WARPS);
@@ -141,7 +148,7 @@ IB_EXPORT int ib_paged_attention_generic(const void* q, const void* k_pages, con
     ib_launch(paged_attention_generic_kernel<DPL, JOINT>, grid, 32 * ATT_WARPS, smem, stream,                   \
         (const act_t*)q, (const act_t*)k_pages, (const act_t*)v_pages, block_table, max_pages, page_size,       \
         n_pages, row_request, positions, n_heads, n_kv_heads, head_dim, v_dim, scale, window, (act_t*)out,      \
-        dist_bias, bias_len, head_scale, slopes, sinks)
+        dist_bias, bias_len, opt)
 #define IB_LAUNCH_ATT(DPL) do { if (joint) IB_LAUNCH_ATT_J(DPL, true); else IB_LAUNCH_ATT_J(DPL, false); } while (0)
     if (v_dim <= 32) IB_LAUNCH_ATT(1);
     else if (v_dim <= 64) IB_LAUNCH_ATT(2);

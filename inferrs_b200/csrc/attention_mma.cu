@@ -12,9 +12,11 @@
 //                  (unnormalised sums, row maxima, row sums) go to scratch and a second kernel merges them.
 // A row at position p sees keys lo..p of its request, lo = 0 or p - window + 1.
 //
-// Three options, each a number per head (absent: not applied): head_scale[h] multiplies head h's scaled score,
-// slopes[h] * (p - j) is taken off it, and exp(sinks[h]) joins the softmax's denominator once per row (a place
-// without key and value; with the keys cut over several CTAs it is added where the parts are merged).
+// Options (IbScoreOptions): a factor, a slope and a sink per head, a cap on the scores, a sequence's first keys beside
+// the window, a gate per head.  With the keys cut over several CTAs sink and gate come where the parts are merged.
+//
+// Head sizes are multiples of 16; a row of a tile in shared memory starts at a multiple of 64 elements, so that its
+// 16-byte places can be exchanged by the row's low three bits.
 #include "common.cuh"
 
 #if IB_ACT_BF16
@@ -51,9 +53,11 @@ __device__ __forceinline__ unsigned am_pack(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<unsigned*>(&v);
 }
-// element offset of 16-byte chunk `chunk` of row `row` in a [rows][D] tile whose chunks are XOR-swizzled
+// elements from one row of a tile to the next
+template <int D> __host__ __device__ constexpr int am_pitch() { return (D + 63) / 64 * 64; }
+// element offset of 16-byte chunk `chunk` of row `row` in a tile of heads of D numbers whose chunks are XOR-swizzled
 template <int D> __device__ __forceinline__ int am_swz(int row, int chunk) {
-    return row * D + ((chunk ^ (row & 7)) << 3);
+    return row * am_pitch<D>() + ((chunk ^ (row & 7)) << 3);
 }
 
 struct AttnMmaParams {
@@ -65,14 +69,13 @@ struct AttnMmaParams {
     const int* tile_row0;          // [tiles] first row (token) of the tile
     const int* q_start;            // [R + 1]
     const int* positions;          // [N]
-    __nv_bfloat16* out;            // [N, n_heads * D]
+    __nv_bfloat16* out;            // [N, n_heads * D], rows opt.out_ld apart
     float* part_o;                 // decode form with splits: [N, n_heads, splits, D]
     float* part_ml;                //                          [N, n_heads, splits, 2]
     int max_pages, page_size, n_pages, n_heads, n_kv_heads, window, n_splits;
     float scale_log2;              // scale * log2(e)
-    const float* head_scale;       // [n_heads] or null
-    const float* slopes;           // [n_heads] or null
-    const float* sinks;            // [n_heads] or null
+    float cap_k, cap_c;            // see ib_capped_log2
+    IbScoreOptions opt;
 };
 
 #define AM_LOG2E 1.4426950408889634f
@@ -84,8 +87,9 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
     constexpr int CH = D / 8;  // 16-byte chunks per row
     extern __shared__ __align__(128) unsigned char am_smem[];
     __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(am_smem);
-    __nv_bfloat16* sk = sq + ROWS * D;
-    __nv_bfloat16* sv = sk + ST * AM_KEYS * D;
+    constexpr int PD = am_pitch<D>();
+    __nv_bfloat16* sk = sq + ROWS * PD;
+    __nv_bfloat16* sv = sk + ST * AM_KEYS * PD;
 
     ib_grid_dependency_sync();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -100,12 +104,15 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
     const int p0 = P.positions[row0];
     const int pmax = p0 + n_tok - 1;
     const int lo_min = ib_first_visible(p0, P.window);
-    const int t_first = lo_min / AM_KEYS, t_last = pmax / AM_KEYS + 1;
-    int t_begin = t_first, t_end = t_last;
+    // the tiles that this CTA walks are places i_begin .. i_end - 1 of the list "kept tiles, then the window's"
+    const int keep = P.opt.keep_first;
+    const int t_first = lo_min / AM_KEYS, n_kept = ib_kept_tiles(keep, t_first, AM_KEYS);
+    const int n_all = n_kept + pmax / AM_KEYS + 1 - t_first;
+    int i_begin = 0, i_end = n_all;
     if (DECODE && P.n_splits > 1) {
-        const int per = (t_last - t_first + P.n_splits - 1) / P.n_splits;
-        t_begin = t_first + split * per;
-        t_end = t_begin + per < t_last ? t_begin + per : t_last;
+        const int per = (n_all + P.n_splits - 1) / P.n_splits;
+        i_begin = split * per;
+        i_end = i_begin + per < n_all ? i_begin + per : n_all;
     }
     const int* bt = P.block_table + (long)req * P.max_pages;
 
@@ -119,13 +126,14 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
     }
     am_commit();
 
-    auto load_kv = [&](int t, int buf) {
-        __nv_bfloat16* dk = sk + buf * AM_KEYS * D;
-        __nv_bfloat16* dv = sv + buf * AM_KEYS * D;
+    auto load_kv = [&](int i, int buf) {
+        const int t = ib_nth_tile(i, n_kept, t_first);
+        __nv_bfloat16* dk = sk + buf * AM_KEYS * PD;
+        __nv_bfloat16* dv = sv + buf * AM_KEYS * PD;
         for (int idx = tid; idx < AM_KEYS * CH; idx += AM_THREADS) {
             const int kk = idx / CH, c = idx - kk * CH;
             const int j = t * AM_KEYS + kk;
-            bool valid = j <= pmax && j >= lo_min;
+            bool valid = ib_visible(j, lo_min, pmax, keep);
             int page = 0;
             if (valid) {
                 page = bt[j / P.page_size];
@@ -147,8 +155,8 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
         const int ti = r / G;
         const int head = kvh * G + (r - ti * G);
         const bool head_ok = r - ti * G < G && head < P.n_heads && (DECODE ? r < G : true);
-        scale_r[h] = P.scale_log2 * ((P.head_scale && head_ok) ? P.head_scale[head] : 1.0f);
-        slope_r[h] = (P.slopes && head_ok) ? P.slopes[head] * AM_LOG2E : 0.0f;
+        scale_r[h] = P.scale_log2 * ((P.opt.head_scale && head_ok) ? P.opt.head_scale[head] : 1.0f);
+        slope_r[h] = (P.opt.slopes && head_ok) ? P.opt.slopes[head] * AM_LOG2E : 0.0f;
         if (ti < n_tok) {
             pos_r[h] = p0 + ti;
             lo_r[h] = ib_first_visible(pos_r[h], P.window);
@@ -167,7 +175,7 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
 
 #pragma unroll
     for (int i = 0; i < ST - 1; ++i) {
-        if (t_begin + i < t_end) load_kv(t_begin + i, i);
+        if (i_begin + i < i_end) load_kv(i_begin + i, i);
         am_commit();
     }
     am_wait<ST - 1>();  // the queries have landed
@@ -181,14 +189,15 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
     }
 
     constexpr int NP = DECODE ? 1 : 4;  // pairs of 8-key column tiles that this warp computes per key tile
-    for (int t = t_begin; t < t_end; ++t) {
-        const int buf = (t - t_begin) % ST;
-        if (t + ST - 1 < t_end) load_kv(t + ST - 1, (t + ST - 1 - t_begin) % ST);  // the buffer of tile t - 1
+    for (int it = i_begin; it < i_end; ++it) {
+        const int t = ib_nth_tile(it, n_kept, t_first);
+        const int buf = (it - i_begin) % ST;
+        if (it + ST - 1 < i_end) load_kv(it + ST - 1, (it + ST - 1 - i_begin) % ST);  // the buffer of the tile before
         am_commit();
         am_wait<ST - 1>();
         __syncthreads();
-        const __nv_bfloat16* tk = sk + buf * AM_KEYS * D;
-        const __nv_bfloat16* tv = sv + buf * AM_KEYS * D;
+        const __nv_bfloat16* tk = sk + buf * AM_KEYS * PD;
+        const __nv_bfloat16* tv = sv + buf * AM_KEYS * PD;
 
         float s[2 * NP][4];
 #pragma unroll
@@ -217,8 +226,10 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
             for (int i = 0; i < 4; ++i) {
                 const int h = i >> 1;
                 const int j = t * AM_KEYS + col0 + (i & 1);
-                const bool vis = j >= lo_r[h] && j <= pos_r[h];
-                s[n][i] = vis ? s[n][i] * scale_r[h] - slope_r[h] * (float)(pos_r[h] - j) : -INFINITY;
+                const bool vis = ib_visible(j, lo_r[h], pos_r[h], keep);
+                float x = s[n][i] * scale_r[h] - slope_r[h] * (float)(pos_r[h] - j);
+                if (P.opt.cap > 0.0f) x = ib_capped_log2(x, P.cap_k, P.cap_c);
+                s[n][i] = vis ? x : -INFINITY;
                 mx[h] = fmaxf(mx[h], s[n][i]);
             }
         }
@@ -281,13 +292,14 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
             const int ti = r / G, g = r - ti * G;
             if (ti >= n_tok) continue;
             float inv = l_r[h] > 0.0f ? 1.0f / l_r[h] : 0.0f;
-            if (P.sinks) {     // the place without a key joins the denominator
-                const float sink = P.sinks[kvh * G + g] * AM_LOG2E;
+            if (P.opt.sinks) {     // the place without a key joins the denominator
+                const float sink = P.opt.sinks[kvh * G + g] * AM_LOG2E;
                 const float m_new = fmaxf(m_r[h], sink);
                 const float f = m_r[h] == -INFINITY ? 0.0f : exp2f(m_r[h] - m_new);
                 inv = f / (l_r[h] * f + exp2f(sink - m_new));
             }
-            __nv_bfloat16* dst = P.out + (((long)(row0 + ti) * P.n_heads + kvh * G + g) * D);
+            inv *= ib_head_gate(P.opt, row0 + ti, kvh * G + g);
+            __nv_bfloat16* dst = P.out + (row0 + ti) * P.opt.out_ld + (kvh * G + g) * D;
 #pragma unroll
             for (int n = 0; n < D / 8; ++n) {
                 const __nv_bfloat162 v = __floats2bfloat162_rn(o[n][2 * h] * inv, o[n][2 * h + 1] * inv);
@@ -318,8 +330,8 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
         float M = -INFINITY;
 #pragma unroll
         for (int w = 0; w < 4; ++w) M = fmaxf(M, sm[w * 16 + g]);
-        const bool sink_here = P.sinks != nullptr && P.n_splits == 1;      // with splits the merge kernel adds it
-        const float sink = sink_here ? P.sinks[kvh * G + g] * AM_LOG2E : -INFINITY;
+        const bool sink_here = P.opt.sinks != nullptr && P.n_splits == 1;      // with splits the merge kernel adds it
+        const float sink = sink_here ? P.opt.sinks[kvh * G + g] * AM_LOG2E : -INFINITY;
         M = fmaxf(M, sink);
         float acc = 0.0f, L = 0.0f;
         if (M > -INFINITY) {
@@ -339,22 +351,26 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
                 P.part_ml[(head * P.n_splits + split) * 2 + 1] = L;
             }
         } else {
-            P.out[head * D + e] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
+            P.out[row0 * P.opt.out_ld + (kvh * G + g) * D + e] =
+                __float2bfloat16_rn(L > 0.0f ? acc / L * ib_head_gate(P.opt, row0, kvh * G + g) : 0.0f);
         }
     }
 }
 
 // out[row, head, :] = sum_s 2^(m_s - M) o_s / sum_s 2^(m_s - M) l_s
 __global__ void attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                       __nv_bfloat16* __restrict__ out, int n_splits, int head_dim,
-                                       const float* __restrict__ sinks, int n_heads) {
+                                       __nv_bfloat16* __restrict__ out, int n_splits, int head_dim, int n_heads,
+                                       const IbScoreOptions opt) {
     ib_grid_dependency_sync();
     const long head = blockIdx.x;  // row * n_heads + head
+    const long row = head / n_heads;
+    const int h = (int)(head - row * n_heads);
     const float* ml = part_ml + head * n_splits * 2;
     float M = -INFINITY;
     for (int s = 0; s < n_splits; ++s) M = fmaxf(M, ml[2 * s]);
-    const float sink = sinks ? sinks[head % n_heads] * AM_LOG2E : -INFINITY;
+    const float sink = opt.sinks ? opt.sinks[h] * AM_LOG2E : -INFINITY;
     M = fmaxf(M, sink);
+    const float gate = ib_head_gate(opt, row, h);
     for (int e = threadIdx.x; e < head_dim; e += blockDim.x) {
         float acc = 0.0f, L = 0.0f;
         if (M > -INFINITY) {
@@ -363,9 +379,9 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_o, const f
                 acc += f * part_o[(head * n_splits + s) * head_dim + e];
                 L += f * ml[2 * s + 1];
             }
-            if (sinks) L += exp2f(sink - M);
+            if (opt.sinks) L += exp2f(sink - M);
         }
-        out[head * head_dim + e] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
+        out[row * opt.out_ld + (long)h * head_dim + e] = __float2bfloat16_rn(L > 0.0f ? acc / L * gate : 0.0f);
     }
 }
 
@@ -373,7 +389,7 @@ template <int D, bool DECODE>
 static int launch_attention_mma(const AttnMmaParams& P, int n_tiles, cudaStream_t stream) {
     constexpr int ROWS = DECODE ? 16 : 64;
     constexpr int ST = DECODE ? AM_DECODE_STAGES : 2;
-    const size_t smem = (size_t)(ROWS * D + 2 * ST * AM_KEYS * D) * sizeof(__nv_bfloat16);
+    const size_t smem = (size_t)(ROWS + 2 * ST * AM_KEYS) * am_pitch<D>() * sizeof(__nv_bfloat16);
     static IbDeviceSet configured;   // the attribute is kept per device
     if (const int e = ib_allow_dynamic_smem(configured, paged_attention_mma_kernel<D, DECODE>, smem)) return e;
     const dim3 grid(n_tiles, P.n_kv_heads, DECODE ? P.n_splits : 1);
@@ -387,13 +403,15 @@ IB_EXPORT int ib_paged_attention_mma(const void* q, const void* k_pages, const v
                                      const int* tile_row0, int n_tiles, const int* q_start, const int* positions,
                                      int n_rows, int n_heads, int n_kv_heads, int head_dim, float scale, int window,
                                      void* out, int decode_form, int n_splits, float* part_o, float* part_ml,
-                                     const float* head_scale, const float* slopes, const float* sinks,
-                                     cudaStream_t stream) {
+                                     const float* head_scale, const float* slopes, const float* sinks, float cap,
+                                     int keep_first, const void* gate, long gate_ld, long out_ld, cudaStream_t stream) {
     if (n_tiles <= 0) return IB_OK;
     if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads || page_size <= 0 || max_pages <= 0)
         return IB_ERR_ARGUMENT;
     const int G = n_heads / n_kv_heads;
-    if ((head_dim != 64 && head_dim != 128 && head_dim != 256) || AM_KEYS % page_size || G > 16) return IB_ERR_UNSUPPORTED;
+    if (AM_KEYS % page_size || G > 16) return IB_ERR_UNSUPPORTED;
+    if (keep_first < 0 || out_ld < (long)n_heads * head_dim || out_ld % 2 || (gate != nullptr && gate_ld < n_heads))
+        return IB_ERR_ARGUMENT;
     if (decode_form && n_splits > 1 && (part_o == nullptr || part_ml == nullptr)) return IB_ERR_ARGUMENT;
     AttnMmaParams P;
     P.q = (const __nv_bfloat16*)q; P.k_pages = (const __nv_bfloat16*)k_pages; P.v_pages = (const __nv_bfloat16*)v_pages;
@@ -402,18 +420,21 @@ IB_EXPORT int ib_paged_attention_mma(const void* q, const void* k_pages, const v
     P.max_pages = max_pages; P.page_size = page_size; P.n_pages = n_pages; P.n_heads = n_heads;
     P.n_kv_heads = n_kv_heads; P.window = window; P.n_splits = decode_form ? (n_splits < 1 ? 1 : n_splits) : 1;
     P.scale_log2 = scale * AM_LOG2E;
-    P.head_scale = head_scale; P.slopes = slopes; P.sinks = sinks;
+    P.cap_k = cap > 0.0f ? 2.0f / cap : 0.0f;      // the scores carry the factor log2(e) already
+    P.cap_c = cap * AM_LOG2E;
+    P.opt = {head_scale, slopes, sinks, cap, keep_first, (const act_t*)gate, gate_ld, out_ld};
     int rc;
 #define IB_AM_CASE(DD)                                                                   \
     if (head_dim == DD)                                                                  \
         rc = decode_form ? launch_attention_mma<DD, true>(P, n_tiles, stream)            \
                          : launch_attention_mma<DD, false>(P, n_tiles, stream);
-    IB_AM_CASE(64) else IB_AM_CASE(128) else IB_AM_CASE(256) else rc = IB_ERR_UNSUPPORTED;
+    IB_AM_CASE(64) else IB_AM_CASE(128) else IB_AM_CASE(256) else IB_AM_CASE(32) else IB_AM_CASE(80) else IB_AM_CASE(96)
+    else IB_AM_CASE(192) else rc = IB_ERR_UNSUPPORTED;
 #undef IB_AM_CASE
     if (rc != IB_OK) return rc;
     if (decode_form && P.n_splits > 1) {
         ib_launch(attention_merge_kernel, n_rows * n_heads, head_dim < 128 ? 64 : 128, 0, stream, (const float*)part_o,
-                  (const float*)part_ml, (__nv_bfloat16*)out, P.n_splits, head_dim, sinks, n_heads);
+                  (const float*)part_ml, (__nv_bfloat16*)out, P.n_splits, head_dim, n_heads, P.opt);
         return ib_launch_status();
     }
     return IB_OK;
@@ -473,7 +494,7 @@ IB_EXPORT int ib_paged_attention_decode_noalloc(const void* q, const void* k_pag
     const int code = ib_paged_attention_mma(q, k_pages, v_pages, block_table, max_pages, page_size, n_pages,
                                             row_request, q_start, n_rows, q_start, positions, n_rows, n_heads,
                                             n_kv_heads, head_dim, scale, window, out, 1, n_splits, part_o, part_ml,
-                                            nullptr, nullptr, nullptr, stream);
+                                            nullptr, nullptr, nullptr, 0.0f, 0, nullptr, 0, (long)n_heads * head_dim, stream);
     if (code == IB_ERR_UNSUPPORTED) return IB_NOALLOC_ERR_UNSUPPORTED;
     if (code == IB_ERR_ARGUMENT) return IB_NOALLOC_ERR_ARGUMENT;
     return code;
@@ -483,7 +504,7 @@ IB_EXPORT const char* ib_paged_attention_decode_noalloc_strerror(int code) {
     switch (code) {
         case 0: return "success";
         case IB_NOALLOC_ERR_UNSUPPORTED:
-            return "sizes not taken: head_dim must be 64, 128 or 256, the page size must divide 64, and at most 16 "
+            return "sizes not taken: head_dim must be 32, 64, 80, 96, 128, 192 or 256, the page size must divide 64, and at most 16 "
                    "query heads may share a key/value head";
         case IB_NOALLOC_ERR_ARGUMENT: return "a size is zero or negative, or heads are not a multiple of kv heads";
         case IB_NOALLOC_ERR_TOO_LARGE:
@@ -497,7 +518,8 @@ IB_EXPORT const char* ib_paged_attention_decode_noalloc_strerror(int code) {
 
 IB_EXPORT int ib_paged_attention_mma(const void*, const void*, const void*, const int*, int, int, int, const int*,
                                      const int*, int, const int*, const int*, int, int, int, int, float, int, void*,
-                                     int, int, float*, float*, const float*, const float*, const float*, cudaStream_t) {
+                                     int, int, float*, float*, const float*, const float*, const float*, float, int,
+                                     const void*, long, long, cudaStream_t) {
     return IB_ERR_UNSUPPORTED;
 }
 

@@ -89,6 +89,7 @@ struct Params {
     __nv_bfloat16* out;       // [N, n_heads * 128]
     int max_pages, page_size, n_pages, n_heads, n_kv_heads, window;
     float scale_log2;
+    IbScoreOptions opt;       // of these the kept keys, the gate and the rows' distance
 };
 
 __global__ void __launch_bounds__(THREADS, 1) attention_pair_kernel(const __grid_constant__ CUtensorMap map_q,
@@ -128,7 +129,9 @@ __global__ void __launch_bounds__(THREADS, 1) attention_pair_kernel(const __grid
     // key tiles that each query tile walks: from the first one that its first token's window reaches (the same
     // for both: the earlier tile's) to the one that holds its last token
     const int lo_min = ib_first_visible(p0, P.window);
-    const int t_begin = lo_min / KEYS;
+    const int keep = P.opt.keep_first;              // the tiles that hold kept keys come before the window's
+    const int t_first = lo_min / KEYS, n_kept = ib_kept_tiles(keep, t_first, KEYS);
+    const int t_begin = t_first - n_kept;
     const int n_tok_t[2] = {n_tok < tpt ? n_tok : tpt, n_tok > tpt ? n_tok - tpt : 0};
     int n_tiles_t[2];
     n_tiles_t[0] = (p0 + n_tok_t[0] - 1) / KEYS + 1 - t_begin;
@@ -171,7 +174,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_pair_kernel(const __grid
         const int pages_per_tile = KEYS / P.page_size;   // at most 16
         auto lookup = [&](int i) -> int {
             if (lane >= pages_per_tile) return 0;
-            const int j = (t_begin + i) * KEYS + lane * P.page_size;
+            const int j = ib_nth_tile(i, n_kept, t_first) * KEYS + lane * P.page_size;
             int page = (j <= pmax && j / P.page_size < P.max_pages) ? bt[j / P.page_size] : -1;
             // No page (beyond the request, or given back): the copy is aimed past the last page, where TMA reads
             // nothing and fills the tile with zeros.  No query sees these keys, but their values are multiplied
@@ -278,7 +281,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_pair_kernel(const __grid
             ok = __all_sync(0xffffffffu, ok);   // the tensor-memory loads and stores below are warp-wide
             if (!ok) break;
             fence_after();
-            const int key0 = (t_begin + i) * KEYS;
+            const int key0 = ib_nth_tile(i, n_kept, t_first) * KEYS;
             // The key tile goes in two halves of 64 keys: the second product starts on the first half's P while the
             // second half's exponentials are computed.
 #pragma unroll 1
@@ -289,13 +292,13 @@ __global__ void __launch_bounds__(THREADS, 1) attention_pair_kernel(const __grid
                 tmem_ld32_issue(s_addr + 64 * h + 32, b);
                 tmem_ld_wait();
                 // a half whose keys this row sees in full needs no comparisons (all but the first and last few)
-                const bool all_visible = kbase >= lo && kbase + 63 <= pos;
+                const bool all_visible = kbase + 63 <= pos && (kbase >= lo || kbase + 63 < keep);
                 if (!all_visible) {
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
                         const int ka = kbase + j, kb = ka + 32;
-                        if (!(ka >= lo && ka <= pos)) a[j] = 0xff800000u;   // -inf: exp2 gives 0
-                        if (!(kb >= lo && kb <= pos)) b[j] = 0xff800000u;
+                        if (!ib_visible(ka, lo, pos, keep)) a[j] = 0xff800000u;   // -inf: exp2 gives 0
+                        if (!ib_visible(kb, lo, pos, keep)) b[j] = 0xff800000u;
                     }
                 }
                 // the row's maximum over the half (four chains of three-input maxima)
@@ -363,8 +366,9 @@ __global__ void __launch_bounds__(THREADS, 1) attention_pair_kernel(const __grid
             ok = __all_sync(0xffffffffu, ok);
             if (ok) {
                 fence_after();
-                const float inv = l > 0.0f ? 1.0f / l : 0.0f;
-                __nv_bfloat16* dst = P.out + ((long)(row0 + t * tpt + ti) * P.n_heads + kvh * G + g) * D;
+                const long row = row0 + t * tpt + ti;
+                const float inv = l > 0.0f ? (row_valid ? ib_head_gate(P.opt, row, kvh * G + g) : 1.0f) / l : 0.0f;
+                __nv_bfloat16* dst = P.out + row * P.opt.out_ld + (kvh * G + g) * D;
 #pragma unroll 1
                 for (int c = 0; c < D; c += 32) {
                     unsigned v[32];
@@ -406,12 +410,16 @@ IB_EXPORT int ib_paged_attention_pair_tcgen05(const void* q, const void* k_pages
                                               const int* block_table, int max_pages, int page_size, int n_pages,
                                               const int* tile_req, const int* tile_row0, int n_tiles, const int* q_start,
                                               const int* positions, int n_rows, int n_heads, int n_kv_heads, int head_dim,
-                                              float scale, int window, void* out, cudaStream_t stream) {
+                                              float scale, int window, void* out, int keep_first, const void* gate,
+                                              long gate_ld, long out_ld, cudaStream_t stream) {
     if (n_tiles <= 0) return IB_OK;
     if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads || page_size <= 0 || max_pages <= 0) return IB_ERR_ARGUMENT;
     const int G = n_heads / n_kv_heads;
     if (head_dim != fp::D || fp::KEYS % page_size || page_size < 8 || G > fp::ROWS) return IB_ERR_UNSUPPORTED;
     if (!(scale > 0.0f)) return IB_ERR_UNSUPPORTED;   // the row maximum is taken before the scale is applied
+    if (keep_first < 0 || out_ld < (long)n_heads * head_dim || out_ld % 8 || ((uintptr_t)out & 15) ||
+        (gate != nullptr && gate_ld < n_heads))
+        return IB_ERR_ARGUMENT;
     sm100::EncodeTiled enc = sm100::encode_fn();
     if (enc == nullptr) return IB_ERR_UNSUPPORTED;
     CUtensorMap mq, mk, mv;
@@ -442,6 +450,7 @@ IB_EXPORT int ib_paged_attention_pair_tcgen05(const void* q, const void* k_pages
     P.positions = positions; P.out = (__nv_bfloat16*)out; P.max_pages = max_pages; P.page_size = page_size;
     P.n_pages = n_pages; P.n_heads = n_heads; P.n_kv_heads = n_kv_heads; P.window = window;
     P.scale_log2 = scale * 1.4426950408889634f;
+    P.opt = {nullptr, nullptr, nullptr, 0.0f, keep_first, (const act_t*)gate, gate_ld, out_ld};
     const size_t smem = 2 * fp::TILE_BYTES + 4 * fp::TILE_BYTES + 20 * 8 + fp::SMEM_SLACK;
     static IbDeviceSet configured;   // the attribute is kept per device
     if (const int e = ib_allow_dynamic_smem(configured, fp::attention_pair_kernel, smem)) return e;
@@ -471,7 +480,7 @@ IB_EXPORT int ib_attention_pair_tcgen05_error_async(int* out, cudaStream_t strea
 
 IB_EXPORT int ib_paged_attention_pair_tcgen05(const void*, const void*, const void*, const int*, int, int, int, const int*,
                                               const int*, int, const int*, const int*, int, int, int, int, float, int, void*,
-                                              cudaStream_t) {
+                                              int, const void*, long, long, cudaStream_t) {
     return IB_ERR_UNSUPPORTED;
 }
 IB_EXPORT int ib_attention_pair_tcgen05_error(int) { return 0; }

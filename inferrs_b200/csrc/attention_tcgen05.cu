@@ -59,22 +59,21 @@ struct Params {
     __nv_bfloat16* out;       // [N, n_heads * 128]
     int max_pages, page_size, n_pages, n_heads, n_kv_heads, window;
     float scale_log2;
-    // the form with a number per head (each array [n_heads] or absent): head h's scaled score is multiplied by
-    // head_scale[h], slopes[h] * (position - key) is taken off it, and exp(sinks[h]) joins the row's sum once
-    const float* head_scale;
-    const float* slopes;
-    const float* sinks;
+    float cap_k, cap_c;       // see ib_capped_log2
+    IbScoreOptions opt;
 };
 
 #define FA_LOG2E 1.4426950408889634f
 
-// PER_HEAD: the scores are brought to their final form (factor, slope, mask) before the row's maximum is taken, so
-// a factor may have any sign; without it the maximum is taken over the raw products and scaled afterwards.
-template <bool PER_HEAD>
+// FORM 1: the scores are brought to their final form (factor, slope, mask) before the row's maximum is taken, so
+// a factor may have any sign; without it (FORM 0) the maximum is taken over the raw products and scaled afterwards.
+// FORM 2: the same as 1 with a cap on the scores.
+template <int FORM>
 __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                const __grid_constant__ CUtensorMap map_k,
                                                                const __grid_constant__ CUtensorMap map_v,
                                                                const Params P) {
+    constexpr bool PER_HEAD = FORM != 0, CAPPED = FORM == 2;
     extern __shared__ __align__(1024) unsigned char raw_smem[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(raw_smem) + 1023) & ~(uintptr_t)1023);
     if (smem - raw_smem > SMEM_SLACK) {   // the tiles would not fit behind a base this far off a 1 KB boundary
@@ -110,8 +109,10 @@ __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_cons
     const int p0 = P.positions[row0];
     const int pmax = p0 + n_tok - 1;
     const int lo_min = ib_first_visible(p0, P.window);
-    const int t_begin = lo_min / KEYS, t_end = pmax / KEYS + 1;   // key tiles
-    const int n_tiles = t_end - t_begin;
+    // key tiles: those that hold kept keys, then the window's from t_first on
+    const int keep = P.opt.keep_first;
+    const int t_first = lo_min / KEYS, n_kept = ib_kept_tiles(keep, t_first, KEYS);
+    const int n_tiles = n_kept + pmax / KEYS + 1 - t_first;
 
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
@@ -145,7 +146,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_cons
         const int pages_per_tile = KEYS / P.page_size;   // at most 16
         auto lookup = [&](int i) -> int {
             if (lane >= pages_per_tile) return 0;
-            const int j = (t_begin + i) * KEYS + lane * P.page_size;
+            const int j = ib_nth_tile(i, n_kept, t_first) * KEYS + lane * P.page_size;
             int page = (j <= pmax && j / P.page_size < P.max_pages) ? bt[j / P.page_size] : -1;
             // No page (beyond the request, or given back): the copy is aimed past the last page, where TMA reads
             // nothing and fills the tile with zeros.  No query sees these keys, but their values are multiplied
@@ -229,11 +230,11 @@ __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_cons
         const int pos = row_valid ? p0 + ti : -1;
         const int lo = row_valid ? ib_first_visible(pos, P.window) : 0;
         float sc2 = P.scale_log2, sl2 = 0.0f, sink2 = -INFINITY;
-        if (PER_HEAD) {
+        if (PER_HEAD && g < G && kvh * G + g < P.n_heads) {
             const int head = kvh * G + g;
-            if (P.head_scale) sc2 *= P.head_scale[head];
-            if (P.slopes) sl2 = P.slopes[head] * FA_LOG2E;
-            if (P.sinks) sink2 = P.sinks[head] * FA_LOG2E;
+            if (P.opt.head_scale) sc2 *= P.opt.head_scale[head];
+            if (P.opt.slopes) sl2 = P.opt.slopes[head] * FA_LOG2E;
+            if (P.opt.sinks) sink2 = P.opt.sinks[head] * FA_LOG2E;
         }
         float o[64];
 #pragma unroll
@@ -257,13 +258,13 @@ __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_cons
             const int s = i & 1;
             if (ok && !mbar_wait(s_full0 + 8 * s, (i >> 1) & 1, 5)) ok = false;
             fence_after();
-            const int key0 = (t_begin + i) * KEYS + ch * 64;
+            const int key0 = ib_nth_tile(i, n_kept, t_first) * KEYS + ch * 64;
             unsigned a[32], b[32];
             tmem_ld32_issue(tmem + lane_addr + s * 128 + ch * 64, a);
             tmem_ld32_issue(tmem + lane_addr + s * 128 + ch * 64 + 32, b);
             tmem_ld_wait();
             // a tile whose 64 keys this row sees in full needs no comparisons (all tiles but the first and last few)
-            const bool all_visible = key0 >= lo && key0 + 63 <= pos;
+            const bool all_visible = key0 + 63 <= pos && (key0 >= lo || key0 + 63 < keep);
             // (four running maxima, and four running sums below: one chain of 64 dependent operations would
             // leave the two warps of a scheduler waiting on each other's latencies)
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -279,10 +280,14 @@ __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_cons
                         float vb = decltype(with_slope)::value
                                        ? fmaf(__uint_as_float(b[j]), sc2, fmaf(sl2, (float)(32 + j), base))
                                        : __uint_as_float(b[j]) * sc2;
+                        if (CAPPED) {
+                            va = ib_capped_log2(va, P.cap_k, P.cap_c);
+                            vb = ib_capped_log2(vb, P.cap_k, P.cap_c);
+                        }
                         if (decltype(with_mask)::value) {
                             const int ka = key0 + j, kb = key0 + 32 + j;
-                            if (!(ka >= lo && ka <= pos)) va = -INFINITY;
-                            if (!(kb >= lo && kb <= pos)) vb = -INFINITY;
+                            if (!ib_visible(ka, lo, pos, keep)) va = -INFINITY;
+                            if (!ib_visible(kb, lo, pos, keep)) vb = -INFINITY;
                         }
                         a[j] = __float_as_uint(va);
                         b[j] = __float_as_uint(vb);
@@ -304,8 +309,8 @@ __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_cons
 #pragma unroll
                 for (int j = 0; j < 32; ++j) {
                     const int ka = key0 + j, kb = key0 + 32 + j;
-                    if (!(ka >= lo && ka <= pos)) a[j] = 0xff800000u;   // -inf
-                    if (!(kb >= lo && kb <= pos)) b[j] = 0xff800000u;
+                    if (!ib_visible(ka, lo, pos, keep)) a[j] = 0xff800000u;   // -inf
+                    if (!ib_visible(kb, lo, pos, keep)) b[j] = 0xff800000u;
                     mx4[j & 3] = fmaxf(mx4[j & 3], fmaxf(__uint_as_float(a[j]), __uint_as_float(b[j])));
                 }
             }
@@ -375,7 +380,8 @@ __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_cons
                 const float f = m == -INFINITY ? 0.0f : ex2(m - m_new);
                 inv = f / (l * f + ex2(sink2 - m_new));
             }
-            __nv_bfloat16* dst = P.out + ((long)(row0 + ti) * P.n_heads + kvh * G + g) * D + ch * 64;
+            inv *= ib_head_gate(P.opt, row0 + ti, kvh * G + g);
+            __nv_bfloat16* dst = P.out + (row0 + ti) * P.opt.out_ld + (kvh * G + g) * D + ch * 64;
 #pragma unroll
             for (int c0 = 0; c0 < 64; c0 += 8) {
                 uint4 w;
@@ -401,19 +407,23 @@ __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_cons
 }  // namespace fa
 
 // Prefill-form attention for head size 128, bfloat16: tile i holds up to 128/G tokens of request tile_req[i]
-// from row tile_row0[i].  Same arguments and results as ib_paged_attention_mma with decode_form = 0 (head_scale,
-// slopes and sinks, [n_heads] each, may be absent: with all three absent the form without them runs).
-static int attention_tcgen05_launch(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
-                                    int max_pages, int page_size, int n_pages, const int* tile_req,
-                                    const int* tile_row0, int n_tiles, const int* q_start, const int* positions,
-                                    int n_rows, int n_heads, int n_kv_heads, int head_dim, float scale, int window,
-                                    void* out, const float* head_scale, const float* slopes, const float* sinks,
-                                    cudaStream_t stream) {
+// from row tile_row0[i].  Same arguments and results as ib_paged_attention_mma with decode_form = 0 (without factor,
+// slope, sink and cap the form without them runs); a row of `out` starts at a multiple of 8 elements.
+IB_EXPORT int ib_paged_attention_tcgen05(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
+                                         int max_pages, int page_size, int n_pages, const int* tile_req,
+                                         const int* tile_row0, int n_tiles, const int* q_start, const int* positions,
+                                         int n_rows, int n_heads, int n_kv_heads, int head_dim, float scale, int window,
+                                         void* out, const float* head_scale, const float* slopes, const float* sinks,
+                                         float cap, int keep_first, const void* gate, long gate_ld, long out_ld,
+                                         cudaStream_t stream) {
     if (n_tiles <= 0) return IB_OK;
     if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads || page_size <= 0 || max_pages <= 0) return IB_ERR_ARGUMENT;
     const int G = n_heads / n_kv_heads;
     if (head_dim != fa::D || fa::KEYS % page_size || page_size < 8 || G > fa::ROWS) return IB_ERR_UNSUPPORTED;
     if (!(scale > 0.0f)) return IB_ERR_UNSUPPORTED;   // the row maximum is taken before the scale is applied
+    if (keep_first < 0 || out_ld < (long)n_heads * head_dim || out_ld % 8 || ((uintptr_t)out & 15) ||
+        (gate != nullptr && gate_ld < n_heads))
+        return IB_ERR_ARGUMENT;
     fa::EncodeTiled enc = fa::encode_fn();
     if (enc == nullptr) return IB_ERR_UNSUPPORTED;
     CUtensorMap mq, mk, mv;
@@ -444,40 +454,21 @@ static int attention_tcgen05_launch(const void* q, const void* k_pages, const vo
     P.positions = positions; P.out = (__nv_bfloat16*)out; P.max_pages = max_pages; P.page_size = page_size;
     P.n_pages = n_pages; P.n_heads = n_heads; P.n_kv_heads = n_kv_heads; P.window = window;
     P.scale_log2 = scale * FA_LOG2E;
-    P.head_scale = head_scale; P.slopes = slopes; P.sinks = sinks;
+    P.cap_k = cap > 0.0f ? 2.0f / cap : 0.0f;      // the scores carry the factor log2(e) already
+    P.cap_c = cap * FA_LOG2E;
+    P.opt = {head_scale, slopes, sinks, cap, keep_first, (const act_t*)gate, gate_ld, out_ld};
     const size_t smem = 7 * fa::TILE_BYTES + 18 * 8 + 4 * 128 * 4 + fa::SMEM_SLACK;
-    static IbDeviceSet configured, configured_per_head;   // the attribute is kept per device
-    if (head_scale != nullptr || slopes != nullptr || sinks != nullptr) {
-        if (const int e = ib_allow_dynamic_smem(configured_per_head, fa::attention_kernel<true>, smem)) return e;
-        ib_launch(fa::attention_kernel<true>, dim3(n_tiles * n_kv_heads), fa::THREADS, smem, stream, mq, mk, mv, P);
-        return ib_launch_status();
-    }
-    if (const int e = ib_allow_dynamic_smem(configured, fa::attention_kernel<false>, smem)) return e;
-    ib_launch(fa::attention_kernel<false>, dim3(n_tiles * n_kv_heads), fa::THREADS, smem, stream, mq, mk, mv, P);
+    static IbDeviceSet configured, configured_per_head, configured_capped;   // the attribute is kept per device
+#define FA_LAUNCH(FORM, SET)                                                                                    \
+    do {                                                                                                        \
+        if (const int e = ib_allow_dynamic_smem(SET, fa::attention_kernel<FORM>, smem)) return e;               \
+        ib_launch(fa::attention_kernel<FORM>, dim3(n_tiles * n_kv_heads), fa::THREADS, smem, stream, mq, mk, mv, P); \
+    } while (0)
+    if (cap > 0.0f) FA_LAUNCH(2, configured_capped);
+    else if (head_scale != nullptr || slopes != nullptr || sinks != nullptr) FA_LAUNCH(1, configured_per_head);
+    else FA_LAUNCH(0, configured);
+#undef FA_LAUNCH
     return ib_launch_status();
-}
-
-IB_EXPORT int ib_paged_attention_tcgen05(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
-                                         int max_pages, int page_size, int n_pages, const int* tile_req,
-                                         const int* tile_row0, int n_tiles, const int* q_start, const int* positions,
-                                         int n_rows, int n_heads, int n_kv_heads, int head_dim, float scale, int window,
-                                         void* out, cudaStream_t stream) {
-    return attention_tcgen05_launch(q, k_pages, v_pages, block_table, max_pages, page_size, n_pages, tile_req, tile_row0,
-                                    n_tiles, q_start, positions, n_rows, n_heads, n_kv_heads, head_dim, scale, window, out,
-                                    nullptr, nullptr, nullptr, stream);
-}
-
-// The same with a factor, a slope and a sink per head (each [n_heads] floats or absent).
-IB_EXPORT int ib_paged_attention_tcgen05_per_head(const void* q, const void* k_pages, const void* v_pages,
-                                                  const int* block_table, int max_pages, int page_size, int n_pages,
-                                                  const int* tile_req, const int* tile_row0, int n_tiles,
-                                                  const int* q_start, const int* positions, int n_rows, int n_heads,
-                                                  int n_kv_heads, int head_dim, float scale, int window, void* out,
-                                                  const float* head_scale, const float* slopes, const float* sinks,
-                                                  cudaStream_t stream) {
-    return attention_tcgen05_launch(q, k_pages, v_pages, block_table, max_pages, page_size, n_pages, tile_req, tile_row0,
-                                    n_tiles, q_start, positions, n_rows, n_heads, n_kv_heads, head_dim, scale, window, out,
-                                    head_scale, slopes, sinks, stream);
 }
 
 IB_EXPORT int ib_attention_tcgen05_error(int reset) {
@@ -500,14 +491,8 @@ IB_EXPORT int ib_attention_tcgen05_error_async(int* out, cudaStream_t stream) {
 
 IB_EXPORT int ib_paged_attention_tcgen05(const void*, const void*, const void*, const int*, int, int, int, const int*,
                                          const int*, int, const int*, const int*, int, int, int, int, float, int, void*,
+                                         const float*, const float*, const float*, float, int, const void*, long, long,
                                          cudaStream_t) {
-    return IB_ERR_UNSUPPORTED;
-}
-
-IB_EXPORT int ib_paged_attention_tcgen05_per_head(const void*, const void*, const void*, const int*, int, int, int,
-                                                  const int*, const int*, int, const int*, const int*, int, int, int, int,
-                                                  float, int, void*, const float*, const float*, const float*,
-                                                  cudaStream_t) {
     return IB_ERR_UNSUPPORTED;
 }
 

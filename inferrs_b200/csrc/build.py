@@ -36,7 +36,7 @@ _CORE_SOURCES = ["elementwise.cu", "qk_rope_store.cu", "attention_generic.cu", "
                  "sample_select.cu", "attention_mma.cu", "attention_tcgen05.cu",
                  "attention_pair_tcgen05.cu", "attention_decode.cu", "streams.cu", "linear_scan.cu",
                  "attention_latent.cu", "state_mixers.cu", "decay_scan.cu", "delta_scan.cu", "gated_blocks.cu", "attention_joint_mma.cu",
-                 "conv_attention.cu", "sandwich_norm.cu"]
+                 "conv_attention.cu", "sandwich_norm.cu", "parallel_blocks.cu"]
 
 # name -> (sources, extra flags, extra link flags)
 LIBRARIES: Dict[str, dict] = {

@@ -48,6 +48,49 @@ __device__ __forceinline__ int ib_first_visible(int pos, int span) {
     return 0;
 }
 
+// Beside its window a token may also see the first `keep` keys of its sequence (keep 0: it does not).  `lo` is the
+// first key of the token's window.
+__device__ __forceinline__ bool ib_visible(int j, int lo, int pos, int keep) {
+    return j <= pos && (j >= lo || j < keep);
+}
+
+// Kernels that walk keys in tiles of `keys` walk the tiles that hold kept keys first and then the window's own, from
+// tile t_first on: how many tiles come before t_first, and which tile the i-th one is.
+__device__ __forceinline__ int ib_kept_tiles(int keep, int t_first, int keys) {
+    const int n = (keep + keys - 1) / keys;
+    return n < t_first ? n : t_first;
+}
+__device__ __forceinline__ int ib_nth_tile(int i, int n_kept, int t_first) {
+    return i < n_kept ? i : t_first + i - n_kept;
+}
+
+// What the attention kernels may be asked to do beside scale, mask and softmax.  Arrays are [n_heads] or absent.
+// head_scale[h] multiplies head h's scaled score; slopes[h] * (pos - j) is taken off it; cap > 0: the score then
+// becomes cap * tanh(score / cap); exp(sinks[h]) joins the softmax's denominator once per row (a place without key and
+// value, which nothing before it touches).  keep_first: see ib_visible.  gate: head h's output of row r is multiplied
+// by sigmoid(gate[r * gate_ld + h]).  A row of the output starts out_ld elements after the row before it.
+struct IbScoreOptions {
+    const float* head_scale;
+    const float* slopes;
+    const float* sinks;
+    float cap;
+    int keep_first;
+    const act_t* gate;
+    long gate_ld;
+    long out_ld;
+};
+
+__device__ __forceinline__ float ib_head_gate(const IbScoreOptions& o, long row, int head) {
+    return o.gate ? 1.0f / (1.0f + expf(-ib_to_float(o.gate[row * o.gate_ld + head]))) : 1.0f;
+}
+
+// The cap for kernels whose scores carry a factor log2(e): cap log2(e) tanh(x / cap) of x = raw * factor, through
+// tanh(y) = 1 - 2 / (1 + e^(2 y)), with k = 2 / cap and c = cap log2(e).  Absolute error about c * 2^-22.
+__device__ __forceinline__ float ib_capped_log2(float x, float k, float c) {
+    const float t = exp2f(x * k);
+    return c - __fdividef(2.0f * c, 1.0f + t);
+}
+
 // 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))
 __device__ __forceinline__ float ib_gelu_tanh(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));

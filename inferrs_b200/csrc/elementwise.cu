@@ -13,31 +13,37 @@ IB_EXPORT void ib_set_pdl(int on) { ib_pdl_enabled = on; }
 
 // ---------------------------------------------------------------------------
 // Embedding: out[row, :] = table[ids[row], :] * scale   (the product is formed in float32; scale 1 for
-// architectures that do not scale their embeddings)
+// architectures that do not scale their embeddings).  `copy` (or null) gets the same rows, for models that come back
+// to them.
 // ---------------------------------------------------------------------------
 template <typename WT>
 __global__ void embedding_gather_kernel(const WT* __restrict__ table, const int* __restrict__ ids,
-                                        float* __restrict__ out, int width, int vocab, float scale) {
+                                        float* __restrict__ out, float* __restrict__ copy, int width, int vocab,
+                                        float scale) {
     ib_grid_dependency_sync();
     const int row = blockIdx.x;
     const int id = ids[row];
     const bool ok = id >= 0 && id < vocab;  // the host refuses such ids before the launch
     const WT* src = table + (size_t)(ok ? id : 0) * width;
     float* dst = out + (size_t)row * width;
-    for (int j = threadIdx.x; j < width; j += blockDim.x) dst[j] = ok ? ib_to_float(src[j]) * scale : 0.0f;
+    for (int j = threadIdx.x; j < width; j += blockDim.x) {
+        const float v = ok ? ib_to_float(src[j]) * scale : 0.0f;
+        dst[j] = v;
+        if (copy) copy[(size_t)row * width + j] = v;
+    }
 }
 
-IB_EXPORT int ib_embedding_gather(const void* table, int table_is_f32, const int* ids, float* out, int n_rows,
+IB_EXPORT int ib_embedding_gather(const void* table, int table_is_f32, const int* ids, float* out, float* copy, int n_rows,
                                   int width, int vocab, float scale, cudaStream_t stream) {
     if (n_rows <= 0) return IB_OK;
     if (width <= 0 || vocab <= 0) return IB_ERR_ARGUMENT;
     const int threads = width >= 1024 ? 256 : 128;
     if (table_is_f32)
-        ib_launch(embedding_gather_kernel<float>, n_rows, threads, 0, stream, (const float*)table, ids, out, width, vocab,
-                  scale);
+        ib_launch(embedding_gather_kernel<float>, n_rows, threads, 0, stream, (const float*)table, ids, out, copy, width,
+                  vocab, scale);
     else
         ib_launch(embedding_gather_kernel<__nv_bfloat16>, n_rows, threads, 0, stream, (const __nv_bfloat16*)table, ids, out,
-                  width, vocab, scale);
+                  copy, width, vocab, scale);
     return ib_launch_status();
 }
 

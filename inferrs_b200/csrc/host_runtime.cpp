@@ -66,6 +66,7 @@ struct Request {
 struct Cache {
     int page_size = 0, max_requests = 0;
     std::vector<int> windows;   // per group, -1: all keys stay visible
+    std::vector<int> keeps;     // per group: how many of a sequence's first keys stay visible beside the window
     std::vector<Pool> pools;
     std::deque<int> free_slots;
     std::unordered_map<int64_t, Request> requests;
@@ -157,7 +158,8 @@ struct Cache {
             if (first_needed <= 0) continue;
             int dead = first_needed / page_size;   // pages 0..dead-1 hold only keys before first_needed
             if (dead > (int)r->tables[g].size()) dead = (int)r->tables[g].size();
-            for (int i = 0; i < dead; ++i) {
+            // the pages that hold a sequence's first `keeps[g]` keys stay
+            for (int i = pages_for(keeps[g]); i < dead; ++i) {
                 int& p = r->tables[g][i];
                 if (p != RELEASED) {
                     if (!pools[g].give_back(p)) return ERR_DOUBLE_FREE;
@@ -226,16 +228,19 @@ struct Cache {
 
 #define IBH_EXPORT extern "C" __attribute__((visibility("default")))
 
-// windows[g] < 0: group g keeps all keys.  Returns nullptr for sizes that make no sense.
-IBH_EXPORT void* ibh_cache_new(int n_groups, const int* windows, const int* n_pages, int page_size, int max_requests) {
+// windows[g] < 0: group g keeps all keys; keeps[g] of a sequence's first keys stay visible beside a window.  Returns
+// nullptr for sizes that make no sense.
+IBH_EXPORT void* ibh_cache_new(int n_groups, const int* windows, const int* keeps, const int* n_pages, int page_size,
+                               int max_requests) {
     if (n_groups <= 0 || page_size <= 0 || max_requests <= 0) return nullptr;
     for (int g = 0; g < n_groups; ++g)
-        if (n_pages[g] <= 0 || windows[g] == 0) return nullptr;
+        if (n_pages[g] <= 0 || windows[g] == 0 || keeps[g] < 0) return nullptr;
     Cache* c = new Cache();
     c->page_size = page_size;
     c->max_requests = max_requests;
     for (int g = 0; g < n_groups; ++g) {
         c->windows.push_back(windows[g] < 0 ? -1 : windows[g]);
+        c->keeps.push_back(keeps[g]);
         c->pools.emplace_back(n_pages[g]);
     }
     for (int s = 0; s < max_requests; ++s) c->free_slots.push_back(s);

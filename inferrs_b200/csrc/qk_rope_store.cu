@@ -3,7 +3,8 @@
 // projection output.
 //
 // Input row layout: [ n_heads*d queries | n_kv_heads*d keys | n_kv_heads*d values ]
-// (or queries only, when the layer reads another entry's cache).
+// (or queries only, when the layer reads another entry's cache; or queries and keys only, when a value is its key as it
+// was projected).  A bias over these columns (float) is added first.
 // Norm, rotation angle tables (float) and the products are all 32-bit; only the
 // stores are act_t.
 #include "common.cuh"
@@ -54,7 +55,8 @@ __global__ void qk_norm_rope_store_kernel(
     const float* __restrict__ cos_table, const float* __restrict__ sin_table, int rot_dim, int interleaved, int table_rows,
     const int* __restrict__ positions, const int* __restrict__ row_request,
     const int* __restrict__ block_table, int max_pages, int page_size, int n_pages,
-    act_t* __restrict__ k_pages, act_t* __restrict__ v_pages, act_t* __restrict__ q_out) {
+    act_t* __restrict__ k_pages, act_t* __restrict__ v_pages, act_t* __restrict__ q_out,
+    const float* __restrict__ bias, int value_is_key) {
     extern __shared__ float smem[];
     ib_grid_dependency_sync();
     const int row = blockIdx.x;
@@ -85,9 +87,11 @@ __global__ void qk_norm_rope_store_kernel(
         if (kind == 2) {
             if (kv_place < 0) continue;
             const int kvh = head - n_heads - n_kv_heads;
-            const act_t* src = qkv + (long)row * row_stride + (long)(n_heads + n_kv_heads) * d + (long)kvh * v_dim;
+            const int col = value_is_key ? (n_heads + kvh) * d : (n_heads + n_kv_heads) * d + kvh * v_dim;
+            const act_t* src = qkv + (long)row * row_stride + col;
             act_t* dst = v_pages + (kv_place + (long)kvh * page_size) * v_dim;
-            for (int j = lane; j < v_dim; j += 32) dst[j] = src[j];
+            for (int j = lane; j < v_dim; j += 32)
+                dst[j] = bias ? ib_from_float<act_t>(ib_to_float(src[j]) + bias[col + j]) : src[j];
             if (clear_tail) {
                 const int behind = (page_size - 1 - pos % page_size) * v_dim;
                 for (int j = lane; j < behind; j += 32) dst[v_dim + j] = ib_from_float<act_t>(0.0f);
@@ -97,7 +101,7 @@ __global__ void qk_norm_rope_store_kernel(
         const act_t* src = qkv + (long)row * row_stride + (long)head * d;
         float ss = 0.0f;
         for (int j = lane; j < d; j += 32) {
-            const float v = ib_to_float(src[j]);
+            const float v = ib_to_float(src[j]) + (bias ? bias[head * d + j] : 0.0f);
             sh[j] = v;
             ss += v * v;
         }
@@ -355,20 +359,145 @@ __global__ void qk_norm_rope_store_d128_wide_kernel(
 }
 #endif
 
+// Values that are the keys as they were projected, sixteen bytes per access: a block per row, an item of work per VEC
+// elements of a head (or per VEC elements of its first half and the VEC that turn with them in its second).  Element i
+// of a head's first rot_dim turns with element i + rot_dim / 2, or (INTERLEAVED) element 2i with 2i + 1.  A key is
+// written turned to its page and as it is to the value's.  No norms.
+struct alignas(16) QrsVec { act_t v[16 / sizeof(act_t)]; };
+
+template <bool INTERLEAVED>
+__global__ void qk_rope_store_shared_kernel(
+    const act_t* __restrict__ qk, long row_stride, int n_heads, int n_kv_heads, int d, const float* __restrict__ bias,
+    const float* __restrict__ cos_table, const float* __restrict__ sin_table, int rot_dim, int table_rows,
+    const int* __restrict__ positions, const int* __restrict__ row_request, const int* __restrict__ block_table,
+    int max_pages, int page_size, int n_pages, act_t* __restrict__ k_pages, act_t* __restrict__ v_pages,
+    act_t* __restrict__ q_out) {
+    constexpr int VEC = 16 / (int)sizeof(act_t);
+    ib_grid_dependency_launch();
+    // the step's description, the tables and the biases are written by no kernel: they are read while the kernel
+    // before this one still runs
+    const int row = blockIdx.x;
+    const int pos = positions[row];
+    if (pos < 0 || (rot_dim > 0 && pos >= table_rows)) { ib_note_row_fault(row); ib_grid_dependency_wait(); return; }
+    const int slot = pos % page_size;
+    long kv_place = -1;
+    {
+        const int req = row_request[row];
+        const int page = pos / page_size < max_pages ? block_table[(long)req * max_pages + pos / page_size] : -1;
+        if (page >= 0 && page < n_pages) kv_place = (long)page * n_kv_heads * page_size + slot;
+    }
+    const bool clear_tail = kv_place >= 0 && ib_last_row_of_request(row_request, row, gridDim.x);
+    const int half = rot_dim / 2;
+    const float* c = cos_table + (long)pos * half;
+    const float* s = sin_table + (long)pos * half;
+    const int turning = INTERLEAVED ? rot_dim / VEC : half / VEC;      // items of a head that turn
+    const int items = turning + (d - rot_dim) / VEC;                    // items of a head
+    ib_grid_dependency_wait();
+    for (int it = threadIdx.x; it < (n_heads + n_kv_heads) * items; it += blockDim.x) {
+        const int head = it / items, k = it - head * items;
+        const bool key = head >= n_heads;
+        if (key && kv_place < 0) continue;
+        const bool turns = k < turning;
+        // elements e0 .. e0 + VEC - 1, and e1 .. in the second half
+        const int e0 = INTERLEAVED || turns ? k * VEC : rot_dim + (k - turning) * VEC;
+        const int e1 = e0 + half;
+        const bool two = !INTERLEAVED && turns;
+        const act_t* src = qk + row * row_stride + head * d;
+        float x[VEC], y[VEC];
+        {
+            const QrsVec a = *reinterpret_cast<const QrsVec*>(src + e0);
+            const QrsVec b = *reinterpret_cast<const QrsVec*>(src + (two ? e1 : e0));
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) {
+                x[j] = ib_to_float(a.v[j]) + (bias ? bias[head * d + e0 + j] : 0.0f);
+                y[j] = ib_to_float(b.v[j]) + (bias && two ? bias[head * d + e1 + j] : 0.0f);
+            }
+        }
+        const long place = (kv_place + (long)(head - n_heads) * page_size) * d;
+        QrsVec o;
+        if (key) {
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) o.v[j] = ib_from_float<act_t>(x[j]);
+            *reinterpret_cast<QrsVec*>(v_pages + place + e0) = o;
+            if (two) {
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) o.v[j] = ib_from_float<act_t>(y[j]);
+                *reinterpret_cast<QrsVec*>(v_pages + place + e1) = o;
+            }
+        }
+        if (turns) {
+            if (INTERLEAVED) {
+#pragma unroll
+                for (int j = 0; j < VEC; j += 2) {
+                    const float cs = c[(e0 + j) >> 1], sn = s[(e0 + j) >> 1], u = x[j], v = x[j + 1];
+                    x[j] = u * cs - v * sn;
+                    x[j + 1] = v * cs + u * sn;
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) {
+                    const float cs = c[e0 + j], sn = s[e0 + j], u = x[j], v = y[j];
+                    x[j] = u * cs - v * sn;
+                    y[j] = v * cs + u * sn;
+                }
+            }
+        }
+        act_t* dst = key ? k_pages + place : q_out + ((long)row * n_heads + head) * d;
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) o.v[j] = ib_from_float<act_t>(x[j]);
+        *reinterpret_cast<QrsVec*>(dst + e0) = o;
+        if (two) {
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) o.v[j] = ib_from_float<act_t>(y[j]);
+            *reinterpret_cast<QrsVec*>(dst + e1) = o;
+        }
+    }
+    if (clear_tail) {
+        QrsVec zero;
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) zero.v[j] = ib_from_float<act_t>(0.0f);
+        const int behind = (page_size - 1 - slot) * d / VEC;      // per head
+        for (int it = threadIdx.x; it < n_kv_heads * behind; it += blockDim.x) {
+            const int g = it / behind, k = it - g * behind;
+            *reinterpret_cast<QrsVec*>(v_pages + (kv_place + 1 + (long)g * page_size) * d + k * VEC) = zero;
+        }
+    }
+}
+
+// bias: float over the columns of qkv (or null).  value_is_key: qkv holds queries and keys; a value is its key before the
+// norm and the rotation (v_dim is then head_dim).
 IB_EXPORT int ib_qk_norm_rope_store(const void* qkv, int row_stride, int n_rows, int n_heads, int n_kv_heads,
                                     int head_dim, int v_dim, int store_kv, const void* q_weight, const void* k_weight,
                                     int weight_is_f32, int norm_flags, float eps, const float* cos_table, const float* sin_table,
                                     int rot_dim, int interleaved, int table_rows, const int* positions, const int* row_request,
                                     const int* block_table, int max_pages, int page_size, int n_pages,
-                                    void* k_pages, void* v_pages, void* q_out, cudaStream_t stream) {
+                                    void* k_pages, void* v_pages, void* q_out, const float* bias, int value_is_key,
+                                    cudaStream_t stream) {
     if (n_rows <= 0) return IB_OK;
     if (head_dim <= 0 || head_dim > 1024 || n_heads <= 0 || rot_dim < 0 || rot_dim > head_dim || (rot_dim & 1))
         return IB_ERR_ARGUMENT;
     if (store_kv && (n_kv_heads <= 0 || page_size <= 0 || max_pages <= 0)) return IB_ERR_ARGUMENT;
     if (rot_dim > 0 && (cos_table == nullptr || sin_table == nullptr || table_rows <= 0)) return IB_ERR_ARGUMENT;
-    if (v_dim <= 0 || v_dim > 1024) return IB_ERR_ARGUMENT;
+    if (v_dim <= 0 || v_dim > 1024 || (value_is_key && (!store_kv || v_dim != head_dim))) return IB_ERR_ARGUMENT;
+    {
+        const int vec = 16 / (int)sizeof(act_t);
+        auto on16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+        if (value_is_key && norm_flags == 0 && head_dim % vec == 0 && rot_dim % (interleaved ? vec : 2 * vec) == 0 &&
+            row_stride % vec == 0 && on16(qkv) && on16(q_out) && on16(k_pages) && on16(v_pages)) {
+            const int items = (n_heads + n_kv_heads) * ((interleaved ? rot_dim : rot_dim / 2) + head_dim - rot_dim) / vec;
+            int threads = (items + 31) / 32 * 32;
+            if (threads > 256) threads = 256;
+#define IB_LAUNCH_SHARED(INTER)                                                                                      \
+    ib_launch(qk_rope_store_shared_kernel<INTER>, n_rows, threads, 0, stream, (const act_t*)qkv, (long)row_stride,   \
+              n_heads, n_kv_heads, head_dim, bias, cos_table, sin_table, rot_dim, table_rows, positions, row_request, \
+              block_table, max_pages, page_size, n_pages, (act_t*)k_pages, (act_t*)v_pages, (act_t*)q_out)
+            if (interleaved) IB_LAUNCH_SHARED(true); else IB_LAUNCH_SHARED(false);
+#undef IB_LAUNCH_SHARED
+            return ib_launch_status();
+        }
+    }
     const size_t smem = (size_t)QRS_WARPS * 2 * head_dim * sizeof(float);
-    const bool plain_norms = v_dim == head_dim && (norm_flags & 4) == 0 &&
+    const bool plain_norms = v_dim == head_dim && (norm_flags & 4) == 0 && bias == nullptr && !value_is_key &&
                              ((norm_flags & 1) != 0) == (q_weight != nullptr) &&
                              (!store_kv || ((norm_flags & 2) != 0) == (k_weight != nullptr));
     const int heads_total = n_heads + (store_kv ? 2 * n_kv_heads : 0);
@@ -410,12 +539,12 @@ IB_EXPORT int ib_qk_norm_rope_store(const void* qkv, int row_stride, int n_rows,
         ib_launch(qk_norm_rope_store_kernel<float>, grid, 32 * QRS_WARPS, smem, stream,
             (const act_t*)qkv, row_stride, n_heads, n_kv_heads, head_dim, v_dim, store_kv, (const float*)q_weight,
             (const float*)k_weight, norm_flags, eps, cos_table, sin_table, rot_dim, interleaved, table_rows, positions, row_request, block_table,
-            max_pages, page_size, n_pages, (act_t*)k_pages, (act_t*)v_pages, (act_t*)q_out);
+            max_pages, page_size, n_pages, (act_t*)k_pages, (act_t*)v_pages, (act_t*)q_out, bias, value_is_key);
     else
         ib_launch(qk_norm_rope_store_kernel<__nv_bfloat16>, grid, 32 * QRS_WARPS, smem, stream,
             (const act_t*)qkv, row_stride, n_heads, n_kv_heads, head_dim, v_dim, store_kv, (const __nv_bfloat16*)q_weight,
             (const __nv_bfloat16*)k_weight, norm_flags, eps, cos_table, sin_table, rot_dim, interleaved, table_rows, positions, row_request,
             block_table,
-            max_pages, page_size, n_pages, (act_t*)k_pages, (act_t*)v_pages, (act_t*)q_out);
+            max_pages, page_size, n_pages, (act_t*)k_pages, (act_t*)v_pages, (act_t*)q_out, bias, value_is_key);
     return ib_launch_status();
 }

@@ -10,9 +10,10 @@
 //   convolution state       the last taps - 1 inputs of every request, after the step
 //   gate, then norm         (y * silu(z)) divided by the root mean square of each of `groups` parts, times w
 //   clamped gate            min(g, c) * sigmoid(s min(g, c)) * (clamp(u, -c, c) + 1)
-//   router                  top-k of logits + bias, softmax over the chosen, as a dense row of weights
+//   router                  the chosen experts' weights as a dense row (router.cuh)
 //   routed gate             silu(g) * u * weight of the column's expert
 #include "common.cuh"
+#include "router.cuh"
 
 __device__ __forceinline__ float sm_silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float sm_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
@@ -467,73 +468,32 @@ IB_EXPORT int ib_gelu_rows(const void* z, void* out, long n, cudaStream_t stream
 
 // ---------------------------------------------------------------------------
 // Router.  logits [rows, ld] float hold n_experts router logits per row (and, with has_shared, one more column:
-// the shared expert's gate).  mode 0: weights[r, e] = softmax over the `top` largest of logits[r, :] + bias among
-// themselves for those experts, 0 for the others (equal logits: the lower index wins).  mode 1: the scores are
-// s = sigmoid(logits + bias), the `top` largest scores are chosen (equal scores: the lower index) and
-// weights[r, e] = s_e / (sum of the chosen scores + 1e-20).  mode 2: the same with the scores s = softmax(logits +
-// bias) over all experts.  Either way the weights are multiplied by `scale`;
-// weights[r, n_experts] = sigmoid(logits[r, n_experts]).  One warp per row.
+// the shared expert's gate); weights [rows, n_experts (+ 1)] get a dense row of the experts' weights, zero for those
+// that are not chosen (router.cuh says how), and sigmoid(logits[r, n_experts]) for the shared one.  One warp per row.
 // ---------------------------------------------------------------------------
-__global__ void router_topk_kernel(const float* __restrict__ logits, long ld, const float* __restrict__ bias,
-                                   int n_experts, int top, int has_shared, float* __restrict__ weights, int n_rows,
-                                   int mode, float scale) {
+__global__ void router_topk_kernel(const float* __restrict__ logits, long ld, float* __restrict__ weights, int n_rows,
+                                   const IbRouter R) {
+    extern __shared__ float router_s[];
     ib_grid_dependency_sync();
-    const int lane = threadIdx.x & 31;
-    const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int warp = threadIdx.x >> 5;
+    const int row = blockIdx.x * (blockDim.x >> 5) + warp;
     if (row >= n_rows) return;
-    const float* z = logits + (long)row * ld;
-    float* w = weights + (long)row * (n_experts + has_shared);
-    // a chosen expert is marked by a weight of -1 until the softmax replaces it
-    for (int e = lane; e < n_experts; e += 32) w[e] = 0.0f;
-    __syncwarp();
-    float first = 0.0f, sum = 0.0f;
-    float z_max = -INFINITY, z_den = 1.0f;      // mode 2: the softmax over all experts
-    if (mode == 2) {
-        for (int e = lane; e < n_experts; e += 32) z_max = fmaxf(z_max, z[e] + (bias ? bias[e] : 0.0f));
-        z_max = ib_warp_max(z_max);
-        float d = 0.0f;
-        for (int e = lane; e < n_experts; e += 32) d += expf(z[e] + (bias ? bias[e] : 0.0f) - z_max);
-        z_den = ib_warp_sum(d);
-    }
-    for (int k = 0; k < top; ++k) {
-        float best = -INFINITY;
-        int at = 0x7fffffff;
-        for (int e = lane; e < n_experts; e += 32) {
-            float v = z[e] + (bias ? bias[e] : 0.0f);
-            if (mode == 1) v = sm_sigmoid(v);
-            if (mode == 2) v = expf(v - z_max) / z_den;
-            if (w[e] == 0.0f && (v > best || (v == best && e < at))) { best = v; at = e; }
-        }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-            if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
-        }
-        if (at == 0x7fffffff) break;        // fewer experts than `top`, or nothing but NaN
-        if (k == 0) first = best;
-        sum += mode != 0 ? best : expf(best - first);
-        if (lane == 0) w[at] = -1.0f;
-        __syncwarp();
-    }
-    for (int e = lane; e < n_experts; e += 32)
-        if (w[e] < 0.0f) {
-            const float v = z[e] + (bias ? bias[e] : 0.0f);
-            w[e] = (mode == 1 ? sm_sigmoid(v) / (sum + 1e-20f)
-                    : mode == 2 ? expf(v - z_max) / z_den / (sum + 1e-20f) : expf(v - first) / sum) * scale;
-        }
-    if (has_shared && lane == 0) w[n_experts] = sm_sigmoid(z[n_experts]);
+    ib_route_row(logits + (long)row * ld, router_s + warp * ib_router_scratch(R.n_experts),
+                 weights + (long)row * (R.n_experts + R.has_shared), R);
 }
 
-IB_EXPORT int ib_router_topk(const float* logits, long ld, const float* bias, int n_experts, int top, int has_shared,
-                             float* weights, int n_rows, int mode, float scale, cudaStream_t stream) {
+// bias is added to the logits, correction to the scores by which experts are chosen ([n_experts] each or absent);
+// groups 0: no groups.
+IB_EXPORT int ib_router_topk(const float* logits, long ld, const float* bias, const float* correction, int n_experts,
+                             int top, int has_shared, int groups, int keep, float* weights, int n_rows, int mode,
+                             float scale, cudaStream_t stream) {
     if (n_rows <= 0) return IB_OK;
-    if (n_experts <= 0 || top <= 0 || top > n_experts || logits == nullptr || weights == nullptr || mode < 0 || mode > 2 ||
-        ld < n_experts + (has_shared ? 1 : 0))
-        return IB_ERR_ARGUMENT;
-    const int warps = 4;
-    ib_launch(router_topk_kernel, (n_rows + warps - 1) / warps, 32 * warps, 0, stream, logits, ld, bias, n_experts, top,
-              has_shared ? 1 : 0, weights, n_rows, mode, scale);
+    const IbRouter R = {bias, correction, n_experts, top, has_shared ? 1 : 0, mode, groups, keep, scale};
+    if (!ib_router_ok(R) || logits == nullptr || weights == nullptr || ld < n_experts + R.has_shared) return IB_ERR_ARGUMENT;
+    const int bytes = ib_router_scratch(n_experts) * (int)sizeof(float);
+    const int warps = 4 * bytes <= 40 * 1024 ? 4 : 1;
+    ib_launch(router_topk_kernel, (n_rows + warps - 1) / warps, 32 * warps, (size_t)warps * bytes, stream, logits, ld,
+              weights, n_rows, R);
     return ib_launch_status();
 }
 
@@ -543,9 +503,9 @@ IB_EXPORT int ib_router_topk(const float* logits, long ld, const float* bias, in
 // (e(j) = n_experts).  A token's columns of experts that it did not choose become zero, so the product with the
 // down matrices of all experts, side by side along its inner dimension, is the weighted sum over the chosen.
 // ---------------------------------------------------------------------------
-__global__ void routed_gate_kernel(const act_t* __restrict__ gate_up, const float* __restrict__ weights, int n_weights,
-                                   int n_experts, int ff, act_t* __restrict__ out, int inner, long total, int act_mode,
-                                   float limit, float slope) {
+__global__ void routed_gate_kernel(const act_t* __restrict__ gate_up, long ld_in, const float* __restrict__ weights,
+                                   int n_weights, int n_experts, int ff, act_t* __restrict__ out, long ld_out, int inner,
+                                   long total, int act_mode, float limit, float slope) {
     ib_grid_dependency_sync();
     for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
         const long r = i / inner;
@@ -555,19 +515,19 @@ __global__ void routed_gate_kernel(const act_t* __restrict__ gate_up, const floa
         const float wt = weights[r * n_weights + e];
         float v = 0.0f;
         if (wt != 0.0f) {
-            v = sm_gate_value(act_mode, ib_to_float(gate_up[r * 2 * inner + j]),
-                              ib_to_float(gate_up[r * 2 * inner + inner + j]), limit, slope) * wt;
+            v = sm_gate_value(act_mode, ib_to_float(gate_up[r * ld_in + j]), ib_to_float(gate_up[r * ld_in + inner + j]),
+                              limit, slope) * wt;
         }
-        out[i] = ib_from_float<act_t>(v);
+        out[r * ld_out + j] = ib_from_float<act_t>(v);
     }
 }
 
 // The same, sixteen bytes per thread and one row per blockIdx.y: for expert sizes that are multiples of that many
 // elements (a thread's elements then belong to one expert).  The columns of an expert that the token did not
 // choose are not read.
-__global__ void routed_gate_vec_kernel(const act_t* __restrict__ gate_up, const float* __restrict__ weights,
-                                       int n_weights, int n_experts, int ff, act_t* __restrict__ out, int inner,
-                                       int act_mode, float limit, float slope) {
+__global__ void routed_gate_vec_kernel(const act_t* __restrict__ gate_up, long ld_in, const float* __restrict__ weights,
+                                       int n_weights, int n_experts, int ff, act_t* __restrict__ out, long ld_out,
+                                       int inner, int act_mode, float limit, float slope) {
     ib_grid_dependency_sync();
     const int j = blockIdx.x * blockDim.x + threadIdx.x;
     if (j >= inner / SM_VEC) return;
@@ -577,8 +537,8 @@ __global__ void routed_gate_vec_kernel(const act_t* __restrict__ gate_up, const 
     const float wt = weights[r * n_weights + e];
     SmActVec o;
     if (wt != 0.0f) {
-        const SmActVec g = reinterpret_cast<const SmActVec*>(gate_up + r * 2 * inner)[j];
-        const SmActVec u = reinterpret_cast<const SmActVec*>(gate_up + r * 2 * inner + inner)[j];
+        const SmActVec g = reinterpret_cast<const SmActVec*>(gate_up + r * ld_in)[j];
+        const SmActVec u = reinterpret_cast<const SmActVec*>(gate_up + r * ld_in + inner)[j];
 #pragma unroll
         for (int k = 0; k < SM_VEC; ++k)
             o.v[k] = ib_from_float<act_t>(sm_gate_value(act_mode, ib_to_float(g.v[k]), ib_to_float(u.v[k]), limit,
@@ -587,33 +547,35 @@ __global__ void routed_gate_vec_kernel(const act_t* __restrict__ gate_up, const 
 #pragma unroll
         for (int k = 0; k < SM_VEC; ++k) o.v[k] = ib_from_float<act_t>(0.0f);
     }
-    reinterpret_cast<SmActVec*>(out + r * inner)[j] = o;
+    reinterpret_cast<SmActVec*>(out + r * ld_out)[j] = o;
 }
 
-// clamped != 0: the experts' activation is the clamped form with `limit` and `slope` instead of silu(g) * u.
-IB_EXPORT int ib_routed_gate(const void* gate_up, const float* weights, int n_weights, int n_experts, int ff, void* out,
-                             int n_rows, int inner, int clamped, float limit, float slope, cudaStream_t stream) {
+// Rows of gate_up start ld_in elements apart, rows of out ld_out.  clamped != 0: the experts' activation is the clamped form with `limit` and `slope` instead of silu(g) * u.
+IB_EXPORT int ib_routed_gate(const void* gate_up, long ld_in, const float* weights, int n_weights, int n_experts, int ff,
+                             void* out, long ld_out, int n_rows, int inner, int clamped, float limit, float slope,
+                             cudaStream_t stream) {
     if (n_rows <= 0) return IB_OK;
     if (clamped && !(limit > 0.0f)) return IB_ERR_ARGUMENT;
     const int act_mode = clamped ? 0 : 2;
     if (inner <= 0 || ff <= 0 || n_experts <= 0 || (long)n_experts * ff > inner || weights == nullptr ||
-        n_weights < n_experts + ((long)n_experts * ff < inner ? 1 : 0))
+        n_weights < n_experts + ((long)n_experts * ff < inner ? 1 : 0) || ld_in < 2L * inner || ld_out < inner)
         return IB_ERR_ARGUMENT;
-    if (ff % SM_VEC == 0 && inner % SM_VEC == 0 && sm_aligned16(gate_up) && sm_aligned16(out)) {
+    if (ff % SM_VEC == 0 && inner % SM_VEC == 0 && ld_in % SM_VEC == 0 && ld_out % SM_VEC == 0 && sm_aligned16(gate_up) &&
+        sm_aligned16(out)) {
         const int nv = inner / SM_VEC;
         const int threads = nv >= 256 ? 256 : ((nv + 31) / 32) * 32;
         for (int r0 = 0; r0 < n_rows; r0 += 65535) {   // blockIdx.y holds at most 65,535 rows
             const int rows = n_rows - r0 < 65535 ? n_rows - r0 : 65535;
             ib_launch(routed_gate_vec_kernel, dim3((nv + threads - 1) / threads, rows), threads, 0, stream,
-                      (const act_t*)gate_up + (long)r0 * 2 * inner, weights + (long)r0 * n_weights, n_weights, n_experts,
-                      ff, (act_t*)out + (long)r0 * inner, inner, act_mode, limit, slope);
+                      (const act_t*)gate_up + r0 * ld_in, ld_in, weights + (long)r0 * n_weights, n_weights, n_experts,
+                      ff, (act_t*)out + r0 * ld_out, ld_out, inner, act_mode, limit, slope);
         }
         return ib_launch_status();
     }
     const long total = (long)n_rows * inner;
     long blocks = (total + 255) / 256;
     if (blocks > 148L * 16) blocks = 148L * 16;
-    ib_launch(routed_gate_kernel, (int)blocks, 256, 0, stream, (const act_t*)gate_up, weights, n_weights, n_experts, ff,
-              (act_t*)out, inner, total, act_mode, limit, slope);
+    ib_launch(routed_gate_kernel, (int)blocks, 256, 0, stream, (const act_t*)gate_up, ld_in, weights, n_weights, n_experts,
+              ff, (act_t*)out, ld_out, inner, total, act_mode, limit, slope);
     return ib_launch_status();
 }

@@ -14,7 +14,7 @@ import torch
 
 from .. import kernels
 from ..cache.storage import KVNeed, StateNeed
-from ..parts.basic import Linear, NoNorm, SandwichUpdate
+from ..parts.basic import Linear, NoNorm, SandwichUpdate, SumUpdate
 from ..parts.blocks import BuiltSubLayer, depth_planes
 from ..parts.registry import part_class
 from ..parts.spec import ModelSpec, TensorDecl
@@ -87,6 +87,14 @@ def check_schedule(spec: ModelSpec):
     for i, e in enumerate(spec.schedule):
         if not 0 <= e.layer < len(spec.layers):
             raise ModelError(f"schedule entry {i} names layer {e.layer}; the model has {len(spec.layers)}")
+        if e.add_embedding:
+            first = spec.layers[e.layer].sublayers[0].norm if spec.layers[e.layer].sublayers else None
+            if spec.streams is not None or spec.position_table is not None or spec.embedding_norm is not None or averages \
+                    or spec.layers[e.layer].arrangement not in ("sequential", "parallel") \
+                    or getattr(first, "kind", None) != "rms" or getattr(first, "groups", 1) != 1:
+                raise ModelError(f"schedule entry {i} adds the embedding before layer {e.layer}: that layer starts with a "
+                                 f"plain RMS norm, in a sequential or a parallel block, on a residual of one stream that "
+                                 f"starts from the plain embedding")
         average = spec.layers[e.layer].depth_average
         if averages and (average is None or average.results != i + 2):
             raise ModelError(f"schedule entry {i} runs layer {e.layer}: with averages over depth every layer averages the "
@@ -198,6 +206,7 @@ class Model:
         if self.depth_planes:
             if spec.streams is not None or spec.position_table is not None or spec.embedding_norm is not None:
                 raise ModelError("averages over depth start from the plain embedding on a residual of one stream")
+        self.embedding_again = any(e.add_embedding for e in spec.schedule)
         self._takes_after = ["after" in inspect.signature(b.forward).parameters for b in self.blocks]
         self.embedding_norm = None
         if spec.embedding_norm is not None:
@@ -228,7 +237,9 @@ class Model:
             pending = SandwichUpdate(None, source=planes[0])
         elif self.spec.streams is None and self.position_table is None:
             residual = torch.empty((n, self.spec.width), dtype=torch.float32, device=self.rt.device)
-            kernels.embedding_gather(self.embedding, ctx.token_ids, residual, self.rt.dtype, scale)
+            again = torch.empty_like(residual) if self.embedding_again else None     # for the passes that add it again
+            kernels.embedding_gather(self.embedding, ctx.token_ids, residual, self.rt.dtype, scale,
+                                     **({} if again is None else {"copy": again}))
         else:
             # a residual of several streams [rows, streams, width], each the embedding (plus the position's vector)
             residual = torch.empty((n, self.spec.streams or 1, self.spec.width), dtype=torch.float32,
@@ -243,9 +254,14 @@ class Model:
         schedule = self.spec.schedule
         for k, entry in enumerate(schedule):
             block = self.blocks[entry.layer]
+            if entry.add_embedding:
+                u = SumUpdate.of(pending)
+                if u is None:
+                    raise ModelError(f"schedule entry {k}: the embedding joins the stream beside a plain pending output")
+                pending = SumUpdate(u.delta, u.bias, plus=again)
             # a block that wants to know what runs after it (to fold the norm between into the products around it)
             # is told; the last block's output goes to the last norm, which reads a choice of rows
-            if k + 1 < len(schedule) and self._takes_after[entry.layer]:
+            if k + 1 < len(schedule) and self._takes_after[entry.layer] and not schedule[k + 1].add_embedding:
                 after = getattr(self.blocks[schedule[k + 1].layer], "entry", None)
                 pending = block.forward(ctx, entry.cache, residual, pending, after=after() if after else None)
             else:

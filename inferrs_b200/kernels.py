@@ -24,8 +24,11 @@ class KernelError(RuntimeError):
     pass
 
 
+# head_scale, slopes, sinks, cap, keep_first, gate, gate_ld, out_ld (IbScoreOptions in csrc/common.cuh)
+_SCORE_OPTIONS = (c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_long, c_long)
+
 _SIGNATURES = {
-    "ib_embedding_gather": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
+    "ib_embedding_gather": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
     "ib_rms_norm_rows": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_void_p],
     "ib_add_cast": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
     "ib_logit_scale_softcap": [c_void_p, c_long, c_float, c_float, c_void_p],
@@ -36,15 +39,15 @@ _SIGNATURES = {
     "ib_qk_norm_rope_store": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
                               c_float,
                               c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                              c_void_p, c_void_p, c_void_p, c_void_p],
+                              c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
     "ib_paged_attention_generic": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p,
                                    c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p, c_int,
-                                   c_void_p, c_void_p, c_void_p, c_void_p],
+                                   *_SCORE_OPTIONS, c_void_p],
     "ib_gemm_tn_simt": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_long, c_long,
                         c_long, c_void_p],
     "ib_paged_attention_mma": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                                c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_int,
-                               c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
+                               c_void_p, c_void_p, *_SCORE_OPTIONS, c_void_p],
     "ib_joint_attention_mma": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                                c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p,
                                c_int, c_int, c_void_p, c_void_p, c_void_p],
@@ -52,14 +55,11 @@ _SIGNATURES = {
     "ib_joint_attention_mma_rows": [c_int, c_int, c_int, c_int],
     "ib_paged_attention_tcgen05": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p,
                                    c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
-                                   c_void_p],
-    "ib_paged_attention_tcgen05_per_head": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p,
-                                            c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
-                                            c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
+                                   *_SCORE_OPTIONS, c_void_p],
     "ib_attention_tcgen05_error": [c_int],
     "ib_paged_attention_pair_tcgen05": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p,
                                         c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
-                                        c_void_p],
+                                        c_int, c_void_p, c_long, c_long, c_void_p],
     "ib_attention_pair_tcgen05_error": [c_int],
     "ib_row_fault": [c_int],
     "ib_row_fault_async": [c_void_p, c_void_p],
@@ -68,7 +68,7 @@ _SIGNATURES = {
     "ib_attention_decode_error_async": [c_void_p, c_void_p],
     "ib_paged_attention_decode": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int,
                                   c_int, c_int, c_float, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
-                                  c_void_p, c_void_p, c_void_p],
+                                  c_void_p, c_void_p, *_SCORE_OPTIONS, c_void_p],
     "ib_attention_decode_error": [c_int],
     "ib_argmax": [c_void_p, c_void_p, c_int, c_int, c_long, c_void_p, c_void_p],
     "ib_penalties": [c_void_p, c_long, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -104,7 +104,11 @@ _SIGNATURES = {
                             c_void_p],
     "ib_gate_group_norm": [c_void_p, c_void_p, c_long, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
     "ib_clamped_gate": [c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p],
-    "ib_router_topk": [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p],
+    "ib_router_topk": [c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int,
+                       c_float, c_void_p],
+    "ib_sum_norm_route": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_int,
+                          c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                          c_void_p],
     "ib_gated_add_layer_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int,
                                 c_int, c_void_p],
     "ib_gated_rows": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
@@ -113,8 +117,8 @@ _SIGNATURES = {
     "ib_mix_queries": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "ib_delta_scan": [c_void_p, c_long, c_int, c_int, c_int, c_int, c_void_p, c_long, c_void_p, c_long, c_float, c_float,
                       c_void_p, c_long, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
-    "ib_routed_gate": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float, c_float,
-                       c_void_p],
+    "ib_routed_gate": [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_void_p, c_long, c_int, c_int, c_int, c_float,
+                       c_float, c_void_p],
     "ib_decay_scan": [c_void_p, c_long, c_int, c_int, c_int, c_int, c_void_p, c_long, c_void_p, c_long, c_void_p,
                       c_void_p, c_long, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "ib_causal_conv_rows": [c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_void_p, c_long, c_long, c_void_p, c_void_p,
@@ -209,21 +213,33 @@ def _p(t: Optional[torch.Tensor]) -> Optional[int]:
     return None if t is None else t.data_ptr()
 
 
+def _need_rows(t: torch.Tensor, name: str, dtypes) -> int:
+    """Like :func:`_need` for a matrix whose rows may lie apart (columns of a wider one): the distance of two rows."""
+    if not (t.is_cuda and t.dim() == 2 and t.dtype in dtypes and t.stride(1) == 1 and t.stride(0) >= t.shape[1]):
+        raise KernelError(f"{name} must be a CUDA matrix of {dtypes} with rows of neighbouring elements, got {t.dtype} "
+                          f"{tuple(t.shape)} with strides {t.stride()} on {t.device}")
+    return t.stride(0)
+
+
 _W = (torch.float32, torch.bfloat16)
 _I = (torch.int32,)
 
 
 def embedding_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, act_dtype: torch.dtype,
-                     scale: float = 1.0):
-    """out[r, :] = table[ids[r], :] * scale as float32."""
+                     scale: float = 1.0, copy: Optional[torch.Tensor] = None):
+    """out[r, :] = table[ids[r], :] * scale as float32; ``copy`` (float32, like ``out``) gets the same rows."""
+    _need(copy, "copy", (torch.float32,), 2, optional=True)
+    if copy is not None and copy.shape != out.shape:
+        raise KernelError(f"embedding_gather: copy {tuple(copy.shape)}, out {tuple(out.shape)}")
     _need(table, "table", _W, 2)
     _need(ids, "ids", _I, 1)
     _need(out, "out", (torch.float32,), 2)
     n, width = out.shape
     if ids.shape[0] != n or table.shape[1] != width:
         raise KernelError(f"embedding_gather: ids {tuple(ids.shape)}, table {tuple(table.shape)}, out {tuple(out.shape)}")
-    _check(_core(act_dtype).ib_embedding_gather(_p(table), int(table.dtype == torch.float32), _p(ids), _p(out), n,
-                                                width, table.shape[0], float(scale), _stream()), "embedding_gather")
+    _check(_core(act_dtype).ib_embedding_gather(_p(table), int(table.dtype == torch.float32), _p(ids), _p(out),
+                                                _p(copy), n, width, table.shape[0], float(scale), _stream()),
+           "embedding_gather")
 
 
 def embedding_streams(table: torch.Tensor, ids: torch.Tensor, pos_table: Optional[torch.Tensor],
@@ -657,20 +673,23 @@ def qk_norm_rope_store(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_di
                        positions: torch.Tensor, row_request: torch.Tensor, block_table: Optional[torch.Tensor],
                        k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], q_out: torch.Tensor,
                        interleaved: bool = False, norm_q: Optional[bool] = None, norm_k: Optional[bool] = None,
-                       norm_after_rotation: bool = False):
+                       norm_after_rotation: bool = False, bias: Optional[torch.Tensor] = None,
+                       value_is_key: bool = False):
     """Per-head norm of q and k, rotation by position, q to ``q_out``, k and v into their pages.  Element ``i`` of
     a head's first ``rot_dim / 2`` turns with element ``i + rot_dim / 2``; ``interleaved``: element ``2i`` with ``2i + 1``.
 
     ``norm_q`` / ``norm_k`` say whether queries / keys are divided by their root mean square (None: where a weight is
     given); a normed kind without a weight is divided and nothing else.  ``norm_after_rotation``: the norm comes
     after the rotation instead of before it.  Values may have another size than keys (the last size of ``v_pages``).
+    ``bias`` (float32, one number per column of q, k and v) is added first.  ``value_is_key``: there are no value columns;
+    a value is its key as it was projected (with its bias), before norm and rotation.
 
     qkv [N, at least n_heads * d + n_kv_heads * (d + dv)] (queries only when ``store_kv`` is False; columns behind
     them, a gate's for instance, are not read);
     pages [n_pages, n_kv_heads, page_size, d or dv]; block_table int32 [R, max_pages].
     """
     act = q_out.dtype
-    _need(qkv, "qkv", (act,), 2)
+    ld = _need_rows(qkv, "qkv", (act,))
     _need(q_out, "q_out", _W, 3)
     _need(positions, "positions", _I, 1)
     _need(row_request, "row_request", _I, 1)
@@ -679,7 +698,12 @@ def qk_norm_rope_store(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_di
     if store_kv:
         _need(v_pages, "v_pages", (act,), 4)
         v_dim = v_pages.shape[3]
-    cols = n_heads * head_dim + (n_kv_heads * (head_dim + v_dim) if store_kv else 0)
+    if value_is_key and (not store_kv or v_dim != head_dim):
+        raise KernelError("qk_norm_rope_store: values that are keys are stored with them and have their size")
+    cols = n_heads * head_dim + (n_kv_heads * (head_dim + (0 if value_is_key else v_dim)) if store_kv else 0)
+    _need(bias, "bias", (torch.float32,), 1, optional=True)
+    if bias is not None and bias.shape[0] != cols:
+        raise KernelError(f"qk_norm_rope_store: a bias of {bias.shape[0]} numbers for {cols} columns")
     if qkv.shape[1] < cols or q_out.shape != (n, n_heads, head_dim) or positions.shape[0] != n \
             or row_request.shape[0] != n:
         raise KernelError(f"qk_norm_rope_store: qkv {tuple(qkv.shape)} (want {cols} columns), q_out "
@@ -715,11 +739,11 @@ def qk_norm_rope_store(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_di
                               f"{n_kv_heads} heads of {head_dim}")
         max_pages = block_table.shape[1]
     _check(_core(act).ib_qk_norm_rope_store(
-        _p(qkv), qkv.shape[1], n, n_heads, n_kv_heads, head_dim, v_dim, int(store_kv), _p(q_weight), _p(k_weight),
+        _p(qkv), ld, n, n_heads, n_kv_heads, head_dim, v_dim, int(store_kv), _p(q_weight), _p(k_weight),
         int(wdt == torch.float32), flags, float(eps), _p(cos) if rot_dim else None, _p(sin) if rot_dim else None, rot_dim,
         int(bool(interleaved)), table_rows, _p(positions), _p(row_request), _p(block_table) if store_kv else None, max_pages, page_size,
-        n_pages, _p(k_pages) if store_kv else None, _p(v_pages) if store_kv else None, _p(q_out), _stream()),
-        "qk_norm_rope_store")
+        n_pages, _p(k_pages) if store_kv else None, _p(v_pages) if store_kv else None, _p(q_out), _p(bias),
+        int(bool(value_is_key)), _stream()), "qk_norm_rope_store")
 
 
 def row_fault(act_dtype: torch.dtype, reset: bool = True) -> Optional[int]:
@@ -741,34 +765,72 @@ def span_argument(window: Optional[int], chunk: Optional[int] = None) -> int:
     return int(window) if window else (-int(chunk) if chunk else 0)
 
 
+@dataclass
+class ScoreOptions:
+    """What attention may be asked to do beside scale, mask and softmax; every kernel says which of it it takes.
+
+    ``head_scale`` / ``slopes`` / ``sinks``: float32 [H] each.  Head h's scaled score is multiplied by head_scale[h];
+    slopes[h] * (pos - j) is taken off it; every row's softmax gets one more term, exp(sinks[h]), in its denominator
+    only (no key or value belongs to it; scale, factor, slope and cap leave it alone).  ``cap``: the score then becomes
+    cap * tanh(score / cap).  ``keep_first``: beside its window a token sees the first keep_first keys of its sequence.
+    ``gate`` [rows, at least H] in the activation dtype (a view of a wider matrix may be given): head h's output of
+    row r is multiplied by sigmoid(gate[r, h])."""
+
+    head_scale: Optional[torch.Tensor] = None
+    slopes: Optional[torch.Tensor] = None
+    sinks: Optional[torch.Tensor] = None
+    cap: Optional[float] = None
+    keep_first: int = 0
+    gate: Optional[torch.Tensor] = None
+
+    @property
+    def shape_scores(self) -> bool:
+        """Whether the scores or the softmax are changed (not only which keys are seen and what becomes of the output)."""
+        return self.head_scale is not None or self.slopes is not None or self.sinks is not None or self.cap is not None
+
+    def check(self, what: str, n_rows: int, n_heads: int, act: torch.dtype):
+        for name, t in (("head_scale", self.head_scale), ("slopes", self.slopes), ("sinks", self.sinks)):
+            _need(t, name, (torch.float32,), 1, optional=True)
+            if t is not None and t.shape[0] != n_heads:
+                raise KernelError(f"{what}: {name} has {t.shape[0]} numbers for {n_heads} heads")
+        if self.cap is not None and not self.cap > 0:
+            raise KernelError(f"{what}: a cap on the scores is positive, got {self.cap}")
+        if self.keep_first < 0:
+            raise KernelError(f"{what}: keep_first must not be negative, got {self.keep_first}")
+        if self.gate is not None:
+            _need_rows(self.gate, "gate", (act,))
+            if self.gate.shape[0] != n_rows or self.gate.shape[1] < n_heads:
+                raise KernelError(f"{what}: a gate {tuple(self.gate.shape)} for {n_rows} rows of {n_heads} heads")
+
+    def output_args(self):
+        """keep_first, gate, gate_ld"""
+        return (int(self.keep_first), _p(self.gate), 0 if self.gate is None else self.gate.stride(0))
+
+    def args(self):
+        return (_p(self.head_scale), _p(self.slopes), _p(self.sinks), float(self.cap or 0.0)) + self.output_args()
+
+
 def paged_attention_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
                             row_request: torch.Tensor, positions: torch.Tensor, scale: float, window: Optional[int],
-                            out: torch.Tensor, joint: bool = False, dist_bias: Optional[torch.Tensor] = None,
-                            head_scale: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                            sinks: Optional[torch.Tensor] = None):
+                            out: torch.Tensor, joint: bool = False, dist_bias: Optional[torch.Tensor] = None, **options):
     """out[r, h*dv:(h+1)*dv] = attention of token r's head h over its request's cached keys lo..pos.  ``window``:
     see :func:`span_argument` (a negative number: chunks).  Values may have another size dv than keys.
 
     ``joint``: ``q`` is [rows, H, kv_heads * d], one vector per key/value head side by side, and a score is the sum
     of its products with all key heads of the token (the form that queries mixed by :func:`mix_queries` take).
     ``dist_bias`` float32 [H, L]: dist_bias[h, pos - j] is taken off head h's score against key j (a distance beyond
-    the table reads its last entry).
-
-    ``head_scale`` / ``slopes`` / ``sinks``: float32 [H] each.  Head h's scaled score is multiplied by head_scale[h];
-    slopes[h] * (pos - j) is taken off it; every row's softmax gets one more term, exp(sinks[h]), in its denominator
-    only (no key or value belongs to it; scale, factor and slope leave it alone)."""
+    the table reads its last entry).  ``options``: the fields of :class:`ScoreOptions`, all of them.  The rows of ``out``
+    may lie apart."""
     act = out.dtype
+    opt = ScoreOptions(**options)
     _need(q, "q", (act,), 3)
-    for name, t in (("head_scale", head_scale), ("slopes", slopes), ("sinks", sinks)):
-        _need(t, name, (torch.float32,), 1, optional=True)
-        if t is not None and t.shape[0] != q.shape[1]:
-            raise KernelError(f"paged_attention: {name} has {t.shape[0]} numbers for {q.shape[1]} heads")
+    opt.check("paged_attention", q.shape[0], q.shape[1], act)
     _need(k_pages, "k_pages", (act,), 4)
     _need(v_pages, "v_pages", (act,), 4)
     _need(block_table, "block_table", _I, 2)
     _need(row_request, "row_request", _I, 1)
     _need(positions, "positions", _I, 1)
-    _need(out, "out", _W, 2)
+    out_ld = _need_rows(out, "out", _W)
     _need(dist_bias, "dist_bias", (torch.float32,), 2, optional=True)
     n, nh, dq = q.shape
     n_pages, nkv, page_size, dk = k_pages.shape
@@ -784,7 +846,7 @@ def paged_attention_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: tor
     _check(_core(act).ib_paged_attention_generic(
         _p(q), _p(k_pages), _p(v_pages), _p(block_table), block_table.shape[1], page_size, n_pages, _p(row_request),
         _p(positions), n, nh, nkv, d, dv, float(scale), int(window) if window else 0, _p(out), int(bool(joint)),
-        _p(dist_bias), 0 if dist_bias is None else dist_bias.shape[1], _p(head_scale), _p(slopes), _p(sinks), _stream()),
+        _p(dist_bias), 0 if dist_bias is None else dist_bias.shape[1], *opt.args(), out_ld, _stream()),
         "paged_attention_generic")
 
 
@@ -1311,27 +1373,119 @@ def gelu_rows(z: torch.Tensor, out: torch.Tensor):
 ROUTE_SOFTMAX_OF_CHOSEN, ROUTE_SIGMOID_SHARE, ROUTE_SOFTMAX_SHARE = 0, 1, 2
 
 
+@dataclass
+class Router:
+    """How a row's experts are chosen and weighed (csrc/router.cuh).  ``mode`` ROUTE_SOFTMAX_OF_CHOSEN: the ``top``
+    largest logits, weighed by the softmax over themselves.  ROUTE_SIGMOID_SHARE: the scores are sigmoid(logits + bias), the
+    ``top`` largest are chosen and each weighs its score over the sum of the chosen scores (+ 1e-20).
+    ROUTE_SOFTMAX_SHARE: the same with softmax(logits + bias) over all experts.  ``correction`` is added to the scores by
+    which experts are chosen, not to those that weigh.  ``groups`` > 0: the experts form that many equal groups of
+    neighbours, a group's worth is the sum of its two largest choice scores, and only the ``keep`` best groups' experts
+    can be chosen.  The weights are multiplied by ``scale``.  ``has_shared``: one more logit, whose sigmoid is the shared
+    expert's weight.  ``weight`` [n_experts + has_shared, width]: the router's own matrix, where a kernel makes the logits
+    itself."""
+
+    n_experts: int
+    top: int
+    bias: Optional[torch.Tensor] = None
+    correction: Optional[torch.Tensor] = None
+    has_shared: bool = False
+    groups: int = 0
+    keep: int = 0
+    mode: int = 0
+    scale: float = 1.0
+    weight: Optional[torch.Tensor] = None
+
+    @property
+    def columns(self) -> int:
+        return self.n_experts + int(bool(self.has_shared))
+
+    def check(self, what: str):
+        for name, t in (("bias", self.bias), ("correction", self.correction)):
+            _need(t, name, (torch.float32,), 1, optional=True)
+            if t is not None and t.shape[0] != self.n_experts:
+                raise KernelError(f"{what}: {name} has {t.shape[0]} numbers for {self.n_experts} experts")
+        if not 0 < self.top <= self.n_experts or self.n_experts > 2048:
+            raise KernelError(f"{what}: {self.top} of {self.n_experts} experts (at most 2048)")
+        if self.mode not in (ROUTE_SOFTMAX_OF_CHOSEN, ROUTE_SIGMOID_SHARE, ROUTE_SOFTMAX_SHARE):
+            raise KernelError(f"{what}: unknown mode {self.mode}")
+        if self.groups < 0 or (self.groups and (self.n_experts % self.groups or not 0 < self.keep <= self.groups
+                                                or self.keep * (self.n_experts // self.groups) < self.top)):
+            raise KernelError(f"{what}: {self.keep} of {self.groups} groups of {self.n_experts} experts, {self.top} chosen")
+
+
 def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], n_experts: int, top: int, has_shared: bool,
-                weights: torch.Tensor, act_dtype: torch.dtype, mode: int = ROUTE_SOFTMAX_OF_CHOSEN, scale: float = 1.0):
-    """weights[r, e] = the softmax over the ``top`` largest of logits[r, :n_experts] + bias, among themselves, for
-    those experts and 0 for the others; with ``has_shared`` weights[r, n_experts] = sigmoid(logits[r, n_experts]).
-    ``mode`` ROUTE_SIGMOID_SHARE: the scores are sigmoid(logits + bias), the ``top`` largest are chosen and each
-    chosen expert weighs its score over the sum of the chosen scores (+ 1e-20).  ROUTE_SOFTMAX_SHARE: the same with the
-    scores softmax(logits + bias) over all experts.  The routed weights are multiplied by ``scale``."""
+                weights: torch.Tensor, act_dtype: torch.dtype, mode: int = ROUTE_SOFTMAX_OF_CHOSEN, scale: float = 1.0,
+                correction: Optional[torch.Tensor] = None, groups: int = 0, keep: int = 0):
+    """weights[r, e] = the experts' weights of row r by its float32 router logits, 0 for those that are not chosen
+    (:class:`Router` says how); with ``has_shared`` weights[r, n_experts] = sigmoid(logits[r, n_experts])."""
+    r = Router(n_experts=int(n_experts), top=int(top), bias=bias, correction=correction, has_shared=bool(has_shared),
+               groups=int(groups), keep=int(keep), mode=int(mode), scale=float(scale))
+    route(logits, r, weights, act_dtype)
+
+
+def route(logits: torch.Tensor, router: Router, weights: torch.Tensor, act_dtype: torch.dtype):
+    """:func:`router_topk` with the router as one object."""
     _need(logits, "logits", (torch.float32,), 2)
-    _need(bias, "bias", (torch.float32,), 1, optional=True)
     _need(weights, "weights", (torch.float32,), 2)
+    router.check("router_topk")
     n = logits.shape[0]
-    cols = n_experts + int(bool(has_shared))
-    if logits.shape[1] < cols or weights.shape != (n, cols) or (bias is not None and bias.shape[0] != n_experts) \
-            or not 0 < top <= n_experts:
-        raise KernelError(f"router_topk: logits {tuple(logits.shape)}, weights {tuple(weights.shape)}, top {top} of "
-                          f"{n_experts}")
-    if mode not in (ROUTE_SOFTMAX_OF_CHOSEN, ROUTE_SIGMOID_SHARE, ROUTE_SOFTMAX_SHARE):
-        raise KernelError(f"router_topk: unknown mode {mode}")
-    _check(_core(act_dtype).ib_router_topk(_p(logits), logits.shape[1], _p(bias), int(n_experts), int(top),
-                                           int(bool(has_shared)), _p(weights), n, int(mode), float(scale), _stream()),
-           "router_topk")
+    if logits.shape[1] < router.columns or weights.shape != (n, router.columns):
+        raise KernelError(f"router_topk: logits {tuple(logits.shape)}, weights {tuple(weights.shape)}, {router.columns} columns")
+    _check(_core(act_dtype).ib_router_topk(
+        _p(logits), logits.shape[1], _p(router.bias), _p(router.correction), router.n_experts, router.top,
+        int(router.has_shared), router.groups, router.keep, _p(weights), n, router.mode, router.scale, _stream()),
+        "router_topk")
+
+
+SUM_NORM_MAX_WIDTH = 32768          # the row in shared memory (csrc/parallel_blocks.cu)
+SUM_NORM_MAX_SHARED = 200 * 1024    # bytes of row, logits and router scratch
+
+
+def sum_norm_routes(width: int, router: Router) -> bool:
+    """Whether the kernel that norms a row also routes it at these sizes."""
+    up4 = lambda v: (v + 3) // 4 * 4                                                              # noqa: E731
+    return width <= SUM_NORM_MAX_WIDTH and router.n_experts <= 2048 and \
+        4 * (up4(width) + up4(router.columns) + 5 * router.n_experts) <= SUM_NORM_MAX_SHARED
+
+
+def sum_norm_route(residual: torch.Tensor, delta: Optional[torch.Tensor], bias: Optional[torch.Tensor],
+                   plus: Optional[torch.Tensor], weight: torch.Tensor, eps: float, out: torch.Tensor,
+                   rows: Optional[torch.Tensor] = None, router: Optional[Router] = None,
+                   shares: Optional[torch.Tensor] = None):
+    """residual += delta + bias + plus (float32, in place; each may be None: ``delta`` in the activation dtype, ``bias``
+    float32 [width], ``plus`` float32 rows); out = rms_norm(residual) * weight; and with a ``router`` shares[r] = the experts' weights
+    by the logits of the row in ``out``.  With ``rows`` (int32 [W]) only those rows are read, nothing is written back and
+    nothing routed."""
+    act = out.dtype
+    _need(residual, "residual", (torch.float32,), 2)
+    _need(delta, "delta", (act,), 2, optional=True)
+    _need(bias, "bias", (torch.float32,), 1, optional=True)
+    _need(plus, "plus", (torch.float32,), 2, optional=True)
+    _need(weight, "weight", _W, 1)
+    _need(out, "out", _W, 2)
+    _need(rows, "rows", _I, 1, optional=True)
+    n, width = residual.shape
+    n_out = n if rows is None else rows.shape[0]
+    if weight.shape[0] != width or out.shape != (n_out, width) or (delta is not None and delta.shape != residual.shape) \
+            or (bias is not None and bias.shape[0] != width) or (plus is not None and plus.shape != residual.shape) \
+            or width > SUM_NORM_MAX_WIDTH:
+        raise KernelError(f"sum_norm_route: residual {tuple(residual.shape)}, weight {tuple(weight.shape)}, out "
+                          f"{tuple(out.shape)} (at most {SUM_NORM_MAX_WIDTH} columns)")
+    r = router or Router(1, 1)
+    if router is not None:
+        router.check("sum_norm_route")
+        _need(router.weight, "router weight", _W, 2)
+        _need(shares, "shares", (torch.float32,), 2)
+        if router.weight.shape != (router.columns, width) or shares.shape != (n, router.columns) or rows is not None:
+            raise KernelError(f"sum_norm_route: router {tuple(router.weight.shape)}, shares {tuple(shares.shape)} for "
+                              f"{router.columns} columns (and no choice of rows)")
+    w = None if router is None else router.weight
+    _check(_core(act).ib_sum_norm_route(
+        _p(residual), _p(delta), _p(bias), _p(plus), _p(weight), int(weight.dtype == torch.float32), float(eps), _p(out),
+        _p(rows), n_out, width, _p(w), int(w is not None and w.dtype == torch.float32), _p(shares), _p(r.bias),
+        _p(r.correction), r.n_experts, r.top, int(r.has_shared), r.groups, r.keep, r.mode, float(r.scale), _stream()),
+        "sum_norm_route")
 
 
 def routed_gate(gate_up: torch.Tensor, weights: torch.Tensor, n_experts: int, ff: int, out: torch.Tensor,
@@ -1339,18 +1493,18 @@ def routed_gate(gate_up: torch.Tensor, weights: torch.Tensor, n_experts: int, ff
     """out[r, j] = silu(gate_up[r, j]) * gate_up[r, inner + j] * weights[r, e(j)], the experts' columns side by side:
     e(j) = j / ff for the routed ones, n_experts for the columns after them (a shared expert).  With a ``limit`` the
     experts' activation is the clamped form, g sigmoid(slope g) (u + 1) with g = min(gate, limit) and
-    u = clamp(up, -limit, limit), in place of silu(gate) * up."""
+    u = clamp(up, -limit, limit), in place of silu(gate) * up.  The rows of ``gate_up`` and ``out`` may lie apart."""
     act = out.dtype
-    _need(gate_up, "gate_up", (act,), 2)
+    ld_in = _need_rows(gate_up, "gate_up", (act,))
     _need(weights, "weights", (torch.float32,), 2)
-    _need(out, "out", _W, 2)
+    ld_out = _need_rows(out, "out", _W)
     n, inner = out.shape
     if gate_up.shape != (n, 2 * inner) or weights.shape[0] != n or n_experts * ff > inner \
             or weights.shape[1] < n_experts + int(n_experts * ff < inner):
         raise KernelError(f"routed_gate: gate_up {tuple(gate_up.shape)}, weights {tuple(weights.shape)}, out "
                           f"{tuple(out.shape)}")
-    _check(_core(act).ib_routed_gate(_p(gate_up), _p(weights), weights.shape[1], int(n_experts), int(ff), _p(out), n,
-                                     inner, int(limit is not None), float(limit or 0.0), float(slope), _stream()),
+    _check(_core(act).ib_routed_gate(_p(gate_up), ld_in, _p(weights), weights.shape[1], int(n_experts), int(ff), _p(out),
+                                     ld_out, n, inner, int(limit is not None), float(limit or 0.0), float(slope), _stream()),
            "routed_gate")
 
 
@@ -1515,11 +1669,12 @@ def mix_queries(q: torch.Tensor, mix: torch.Tensor, n_kv_heads: int, out: torch.
 
 ARGMAX_CHUNK = 8192      # vocabulary entries per block of the two-stage argmax
 MMA_KEYS = 64          # keys per tile of the tensor-core attention kernel
+MMA_HEAD_DIMS = (32, 64, 80, 96, 128, 192, 256)
 MMA_TARGET_CTAS = 1184  # four waves of 2 resident CTAs on 148 SMs: many small CTAs even out the last wave
 
 
 def mma_attention_supported(dtype: torch.dtype, n_heads: int, n_kv_heads: int, head_dim: int, page_size: int) -> bool:
-    return (dtype == torch.bfloat16 and head_dim in (64, 128, 256) and MMA_KEYS % page_size == 0
+    return (dtype == torch.bfloat16 and head_dim in MMA_HEAD_DIMS and MMA_KEYS % page_size == 0
             and n_heads % n_kv_heads == 0 and n_heads // n_kv_heads <= 16)
 
 
@@ -1534,21 +1689,18 @@ def decode_splits(n_requests: int, n_kv_heads: int, max_kv_len: int) -> int:
 def paged_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
                         tile_req: torch.Tensor, tile_row0: torch.Tensor, n_tiles: int, q_start: torch.Tensor,
                         positions: torch.Tensor, scale: float, window: Optional[int], out: torch.Tensor,
-                        decode_form: bool, n_splits: int = 1, head_scale: Optional[torch.Tensor] = None,
-                        slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None):
+                        decode_form: bool, n_splits: int = 1, **options):
     """Tensor-core attention over the pages (bfloat16).  Prefill form: tile i holds up to 64/G tokens of request
     tile_req[i] from row tile_row0[i].  Decode form: every tile is one token; its keys are cut ``n_splits`` ways
-    and merged through float32 scratch.  ``head_scale`` / ``slopes`` / ``sinks`` (float32 [H]): as in
-    :func:`paged_attention_generic`."""
+    and merged through float32 scratch.  ``options``: the fields of :class:`ScoreOptions`, all of them.  The rows of
+    ``out`` may lie an even number of elements apart."""
     bf = (torch.bfloat16,)
-    for name, t in (("head_scale", head_scale), ("slopes", slopes), ("sinks", sinks)):
-        _need(t, name, (torch.float32,), 1, optional=True)
-        if t is not None and t.shape[0] != q.shape[1]:
-            raise KernelError(f"paged_attention_mma: {name} has {t.shape[0]} numbers for {q.shape[1]} heads")
+    opt = ScoreOptions(**options)
+    opt.check("paged_attention_mma", q.shape[0], q.shape[1], torch.bfloat16)
     _need(q, "q", bf, 3)
     _need(k_pages, "k_pages", bf, 4)
     _need(v_pages, "v_pages", bf, 4)
-    _need(out, "out", bf, 2)
+    out_ld = _need_rows(out, "out", bf)
     for name, t in (("block_table", block_table),):
         _need(t, name, _I, 2)
     for name, t in (("tile_req", tile_req), ("tile_row0", tile_row0), ("q_start", q_start), ("positions", positions)):
@@ -1558,7 +1710,7 @@ def paged_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
     if dk != d or v_pages.shape != k_pages.shape or out.shape != (n, nh * d):
         raise KernelError(f"paged_attention_mma: q {tuple(q.shape)}, pages {tuple(k_pages.shape)}, out {tuple(out.shape)}")
     if not mma_attention_supported(q.dtype, nh, nkv, d, page_size):
-        raise KernelError(f"paged_attention_mma takes head_dim 64/128/256, a page size that divides {MMA_KEYS} and at "
+        raise KernelError(f"paged_attention_mma takes head_dim {MMA_HEAD_DIMS}, a page size that divides {MMA_KEYS} and at "
                           f"most 16 query heads per key/value head; got head_dim {d}, page size {page_size}, "
                           f"{nh}/{nkv} heads")
     if tile_req.shape[0] < n_tiles or tile_row0.shape[0] < n_tiles:
@@ -1570,8 +1722,8 @@ def paged_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
     _check(_core(torch.bfloat16).ib_paged_attention_mma(
         _p(q), _p(k_pages), _p(v_pages), _p(block_table), block_table.shape[1], page_size, n_pages, _p(tile_req),
         _p(tile_row0), n_tiles, _p(q_start), _p(positions), n, nh, nkv, d, float(scale), int(window) if window else 0,
-        _p(out), int(decode_form), int(n_splits), _p(part_o), _p(part_ml), _p(head_scale), _p(slopes), _p(sinks),
-        _stream()), "paged_attention_mma")
+        _p(out), int(decode_form), int(n_splits), _p(part_o), _p(part_ml), *opt.args(), out_ld, _stream()),
+        "paged_attention_mma")
 
 
 _DECODE_COUNTERS = {}  # device index -> zeroed int32 counters of the decode attention kernel
@@ -1617,17 +1769,20 @@ def decode_max_splits(n_requests: int, n_kv_heads: int, max_kv_len: int) -> int:
 def paged_attention_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
                            positions: torch.Tensor, scale: float, window: Optional[int], out: torch.Tensor,
                            max_splits: int, rows: Optional[torch.Tensor] = None, reqs: Optional[torch.Tensor] = None,
-                           min_tiles: int = 4):
+                           min_tiles: int = 4, **options):
     """Attention of one new token per request (row r = request r) over its pages: TMA-fed key/value tiles, split
     over the keys, merged by the slice that finishes last (bfloat16, head_dim 128).  With ``rows`` and ``reqs``
     (int32, equally long) only the rows named are worked on, row ``rows[i]`` being a single token of request
     ``reqs[i]``; a negative row is skipped.  The other rows of ``out`` are left alone.  A request is cut into as
-    many slices as leave each ``min_tiles`` tiles of 64 keys (at most ``max_splits``)."""
+    many slices as leave each ``min_tiles`` tiles of 64 keys (at most ``max_splits``).  ``options``: the fields of
+    :class:`ScoreOptions`, all of them.  The rows of ``out`` may lie a multiple of four elements apart."""
     bf = (torch.bfloat16,)
+    opt = ScoreOptions(**options)
+    opt.check("paged_attention_decode", q.shape[0], q.shape[1], torch.bfloat16)
     _need(q, "q", bf, 3)
     _need(k_pages, "k_pages", bf, 4)
     _need(v_pages, "v_pages", bf, 4)
-    _need(out, "out", bf, 2)
+    out_ld = _need_rows(out, "out", bf)
     _need(block_table, "block_table", _I, 2)
     _need(positions, "positions", _I, 1)
     n_q, nh, d = q.shape
@@ -1657,7 +1812,7 @@ def paged_attention_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torc
     _check(_core(torch.bfloat16).ib_paged_attention_decode(
         _p(q), _p(k_pages), _p(v_pages), _p(block_table), block_table.shape[1], page_size, n_pages, _p(positions), n,
         nh, nkv, d, float(scale), int(window) if window else 0, _p(out), int(max_splits), int(min_tiles), _p(part_o),
-        _p(part_ml), _p(counters), _p(rows), _p(reqs), _stream()), "paged_attention_decode")
+        _p(part_ml), _p(counters), _p(rows), _p(reqs), *opt.args(), out_ld, _stream()), "paged_attention_decode")
 
 
 def attention_decode_error(reset: bool = True) -> int:
@@ -1676,22 +1831,19 @@ def tcgen05_attention_supported(dtype: torch.dtype, n_heads: int, n_kv_heads: in
 
 def paged_attention_tcgen05(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
                             tile_req: torch.Tensor, tile_row0: torch.Tensor, n_tiles: int, q_start: torch.Tensor,
-                            positions: torch.Tensor, scale: float, window: Optional[int], out: torch.Tensor,
-                            head_scale: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                            sinks: Optional[torch.Tensor] = None):
+                            positions: torch.Tensor, scale: float, window: Optional[int], out: torch.Tensor, **options):
     """Attention of prompt portions on tcgen05 tensor cores (bfloat16, head_dim 128): tile i holds up to
     128/G tokens of request tile_req[i] from row tile_row0[i]; Q, K, V by TMA, scores and P V in tensor memory.
-    ``head_scale`` / ``slopes`` / ``sinks`` (float32 [H]): as in :func:`paged_attention_generic`; with any of them the
-    kernel's form runs that brings the scores to their final form before it takes the row's maximum."""
+    ``options``: the fields of :class:`ScoreOptions`, all of them; with a factor, slope, sink or cap the kernel's form
+    runs that brings the scores to their final form before it takes the row's maximum.  The rows of ``out`` may lie a
+    multiple of eight elements apart."""
     bf = (torch.bfloat16,)
-    for name, t in (("head_scale", head_scale), ("slopes", slopes), ("sinks", sinks)):
-        _need(t, name, (torch.float32,), 1, optional=True)
-        if t is not None and t.shape[0] != q.shape[1]:
-            raise KernelError(f"paged_attention_tcgen05: {name} has {t.shape[0]} numbers for {q.shape[1]} heads")
+    opt = ScoreOptions(**options)
+    opt.check("paged_attention_tcgen05", q.shape[0], q.shape[1], torch.bfloat16)
     _need(q, "q", bf, 3)
     _need(k_pages, "k_pages", bf, 4)
     _need(v_pages, "v_pages", bf, 4)
-    _need(out, "out", bf, 2)
+    out_ld = _need_rows(out, "out", bf)
     _need(block_table, "block_table", _I, 2)
     for name, t in (("tile_req", tile_req), ("tile_row0", tile_row0), ("q_start", q_start), ("positions", positions)):
         _need(t, name, _I, 1)
@@ -1702,17 +1854,10 @@ def paged_attention_tcgen05(q: torch.Tensor, k_pages: torch.Tensor, v_pages: tor
     if not tcgen05_attention_supported(q.dtype, nh, nkv, d, page_size):
         raise KernelError(f"paged_attention_tcgen05 takes head_dim 128, a page size of 8..128 that divides 128 and a "
                           f"group size of at most 128; got head_dim {d}, page size {page_size}, {nh}/{nkv} heads")
-    if head_scale is not None or slopes is not None or sinks is not None:
-        _check(_core(torch.bfloat16).ib_paged_attention_tcgen05_per_head(
-            _p(q), _p(k_pages), _p(v_pages), _p(block_table), block_table.shape[1], page_size, n_pages, _p(tile_req),
-            _p(tile_row0), n_tiles, _p(q_start), _p(positions), n, nh, nkv, d, float(scale),
-            int(window) if window else 0, _p(out), _p(head_scale), _p(slopes), _p(sinks), _stream()),
-            "paged_attention_tcgen05")
-        return
     _check(_core(torch.bfloat16).ib_paged_attention_tcgen05(
         _p(q), _p(k_pages), _p(v_pages), _p(block_table), block_table.shape[1], page_size, n_pages, _p(tile_req),
         _p(tile_row0), n_tiles, _p(q_start), _p(positions), n, nh, nkv, d, float(scale), int(window) if window else 0,
-        _p(out), _stream()), "paged_attention_tcgen05")
+        _p(out), *opt.args(), out_ld, _stream()), "paged_attention_tcgen05")
 
 
 TC_PAIR_ROWS = 256  # query rows per tile of the tcgen05 attention kernel with two query tiles per CTA
@@ -1735,16 +1880,21 @@ def tcgen05_pair_attention_supported(dtype: torch.dtype, n_heads: int, n_kv_head
 def paged_attention_pair_tcgen05(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                                  block_table: torch.Tensor, tile_req: torch.Tensor, tile_row0: torch.Tensor, n_tiles: int,
                                  q_start: torch.Tensor, positions: torch.Tensor, scale: float, window: Optional[int],
-                                 out: torch.Tensor):
+                                 out: torch.Tensor, **options):
     """Attention of prompt portions on tcgen05 tensor cores with two query tiles per CTA that take turns
     (bfloat16, head_dim 128): tile i holds up to ``pair_tile_tokens`` tokens of request tile_req[i] from row
     tile_row0[i]; the probabilities go to the second product through tensor memory, where the output is
-    accumulated too."""
+    accumulated too.  Of :class:`ScoreOptions` it takes ``keep_first`` and ``gate``.  The rows of ``out`` may lie a
+    multiple of eight elements apart."""
     bf = (torch.bfloat16,)
+    opt = ScoreOptions(**options)
+    opt.check("paged_attention_pair_tcgen05", q.shape[0], q.shape[1], torch.bfloat16)
+    if opt.shape_scores:
+        raise KernelError("paged_attention_pair_tcgen05 takes no factor, slope, sink or cap on the scores")
     _need(q, "q", bf, 3)
     _need(k_pages, "k_pages", bf, 4)
     _need(v_pages, "v_pages", bf, 4)
-    _need(out, "out", bf, 2)
+    out_ld = _need_rows(out, "out", bf)
     _need(block_table, "block_table", _I, 2)
     for name, t in (("tile_req", tile_req), ("tile_row0", tile_row0), ("q_start", q_start), ("positions", positions)):
         _need(t, name, _I, 1)
@@ -1759,7 +1909,7 @@ def paged_attention_pair_tcgen05(q: torch.Tensor, k_pages: torch.Tensor, v_pages
     _check(_core(torch.bfloat16).ib_paged_attention_pair_tcgen05(
         _p(q), _p(k_pages), _p(v_pages), _p(block_table), block_table.shape[1], page_size, n_pages, _p(tile_req),
         _p(tile_row0), n_tiles, _p(q_start), _p(positions), n, nh, nkv, d, float(scale), int(window) if window else 0,
-        _p(out), _stream()), "paged_attention_pair_tcgen05")
+        _p(out), *opt.output_args(), out_ld, _stream()), "paged_attention_pair_tcgen05")
 
 
 def attention_pair_tcgen05_error(reset: bool = True) -> int:
@@ -1773,78 +1923,64 @@ def attention_tcgen05_error(reset: bool = True) -> int:
 
 
 def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
-                    ctx, scale: float, window: Optional[int], out: torch.Tensor,
-                    head_scale: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                    sinks: Optional[torch.Tensor] = None):
+                    ctx, scale: float, window: Optional[int], out: torch.Tensor, **options):
     """Attention of every row of the step over its request's pages; picks the kernel for the sizes.
 
     ``ctx`` is the step's :class:`~inferrs_b200.engine.batch.StepContext` (row_request, positions
-    and what the faster kernels need to cut the work).  ``head_scale`` / ``slopes`` / ``sinks`` (float32 [H], see
-    :func:`paged_attention_generic`): scores with any of them go to the tcgen05 kernel's per-head form (prompt
-    portions, head size 128), to the ``mma.sync`` kernel (steps of single tokens; head sizes 64 and 256) where these
-    take the sizes, and to the float32 kernel otherwise.
+    and what the faster kernels need to cut the work).  ``options``: the fields of :class:`ScoreOptions`.  Head size
+    128: single tokens run on the TMA decode kernel, prompt portions on the tcgen05 kernels (with a factor, slope, sink or
+    cap on the form that finishes the scores first).  Other head sizes of ``MMA_HEAD_DIMS`` run on the ``mma.sync``
+    kernel, everything else on the float32 kernel.  The rows of ``out`` may lie apart.
     """
+    opt = ScoreOptions(**options)
     n, nh, d = q.shape
     nkv, page_size = k_pages.shape[1], k_pages.shape[2]
-    per_head = dict(head_scale=head_scale, slopes=slopes, sinks=sinks)
-    if v_pages.shape[3] != d or not mma_attention_supported(q.dtype, nh, nkv, d, page_size):
+    if v_pages.shape[3] != d or not mma_attention_supported(q.dtype, nh, nkv, d, page_size) or out.stride(0) % 2 \
+            or out.data_ptr() % 4:
         paged_attention_generic(q, k_pages, v_pages, block_table, ctx.row_request, ctx.positions, scale, window, out,
-                                **per_head)
+                                **options)
         return
-    if any(t is not None for t in per_head.values()):
-        if ctx.decode_only:
-            splits = decode_splits(ctx.n_requests, nkv, min(ctx.max_kv_len, window) if window and window > 0
-                                   else ctx.max_kv_len)
-            paged_attention_mma(q, k_pages, v_pages, block_table, ctx.row_request, ctx.q_start, ctx.n_requests,
-                                ctx.q_start, ctx.positions, scale, window, out, True, splits, **per_head)
-        elif tcgen05_attention_supported(q.dtype, nh, nkv, d, page_size) and scale > 0:
-            # prompt portions (and what single tokens stand beside them) on the tcgen05 kernel's per-head form
-            tile_req, tile_row0, n_tiles = ctx.attention_tiles(TC_ROWS // (nh // nkv))
-            paged_attention_tcgen05(q, k_pages, v_pages, block_table, tile_req, tile_row0, n_tiles, ctx.q_start,
-                                    ctx.positions, scale, window, out, **per_head)
-        else:
-            tile_req, tile_row0, n_tiles = ctx.attention_tiles(MMA_KEYS // (nh // nkv))
-            paged_attention_mma(q, k_pages, v_pages, block_table, tile_req, tile_row0, n_tiles, ctx.q_start,
-                                ctx.positions, scale, window, out, False, **per_head)
+    wide_rows = out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0       # what the TMA kernels' stores need
+    tma_decode = tma_decode_attention_supported(q.dtype, nh, nkv, d, page_size) and wide_rows
+    tcgen05 = tcgen05_attention_supported(q.dtype, nh, nkv, d, page_size) and wide_rows and scale > 0
+    # how many keys a row can reach: what the kernels that cut a row's keys over several CTAs go by
+    reach = min(ctx.max_kv_len, window + opt.keep_first + 2 * MMA_KEYS) if window and window > 0 else ctx.max_kv_len
+    if ctx.decode_only and tma_decode:
+        max_splits, min_tiles = decode_slices(ctx.n_requests, nkv, reach)
+        paged_attention_decode(q, k_pages, v_pages, block_table, ctx.positions, scale, window, out, max_splits,
+                               min_tiles=min_tiles, **options)
+        return
+    if ctx.decode_only:
+        # one row per request: the rows are the tiles
+        paged_attention_mma(q, k_pages, v_pages, block_table, ctx.row_request, ctx.q_start, ctx.n_requests,
+                            ctx.q_start, ctx.positions, scale, window, out, True,
+                            decode_splits(ctx.n_requests, nkv, reach), **options)
+        return
+    if not tcgen05:
+        tile_req, tile_row0, n_tiles = ctx.attention_tiles(MMA_KEYS // (nh // nkv))
+        paged_attention_mma(q, k_pages, v_pages, block_table, tile_req, tile_row0, n_tiles, ctx.q_start,
+                            ctx.positions, scale, window, out, False, **options)
         return
     # Prompt portions: tiles of 256 rows (two query tiles per CTA) where they still give every SM a CTA, else
     # tiles of 128 rows.  A step that stands for a padded one (before its graph is captured) says so.
     pair_tokens = pair_tile_tokens(nh, nkv)
     rows_for_dispatch = ctx.extra.get("dispatch_rows", ctx.n_rows)
-    pair = tcgen05_pair_attention_supported(q.dtype, nh, nkv, d, page_size) \
+    pair = not opt.shape_scores and tcgen05_pair_attention_supported(q.dtype, nh, nkv, d, page_size) \
         and (rows_for_dispatch // pair_tokens) * nkv >= PAIR_MIN_CTAS
     prefill_kernel = paged_attention_pair_tcgen05 if pair else paged_attention_tcgen05
     prefill_tokens = pair_tokens if pair else TC_ROWS // (nh // nkv)
-    if ctx.decode_only and tma_decode_attention_supported(q.dtype, nh, nkv, d, page_size):
-        max_splits, min_tiles = decode_slices(ctx.n_requests, nkv, ctx.max_kv_len)
-        paged_attention_decode(q, k_pages, v_pages, block_table, ctx.positions, scale, window, out, max_splits,
-                               min_tiles=min_tiles)
-    elif ctx.decode_only:
-        # one row per request: the rows are the tiles
-        splits = decode_splits(ctx.n_requests, nkv, ctx.max_kv_len)
-        paged_attention_mma(q, k_pages, v_pages, block_table, ctx.row_request, ctx.q_start, ctx.n_requests,
-                            ctx.q_start, ctx.positions, scale, window, out, True, splits)
-    elif tcgen05_attention_supported(q.dtype, nh, nkv, d, page_size) \
-            and tma_decode_attention_supported(q.dtype, nh, nkv, d, page_size):
+    if tma_decode:
         # portions of prompts and single tokens side by side: the single tokens go to the decode kernel (a tile
         # of the prefill kernel would hold one token of 32), the portions to the prefill kernel
         rows, reqs, n_single = ctx.single_rows()
         if n_single > 0:
-            max_splits, min_tiles = decode_slices(n_single, nkv, ctx.max_kv_len)
+            max_splits, min_tiles = decode_slices(n_single, nkv, reach)
             paged_attention_decode(q, k_pages, v_pages, block_table, ctx.positions, scale, window, out, max_splits,
-                                   rows, reqs, min_tiles=min_tiles)
-        tile_req, tile_row0, n_tiles = ctx.attention_tiles(prefill_tokens, portions_only=True)
-        if n_tiles > 0:
-            prefill_kernel(q, k_pages, v_pages, block_table, tile_req, tile_row0, n_tiles, ctx.q_start,
-                           ctx.positions, scale, window, out)
-    elif tcgen05_attention_supported(q.dtype, nh, nkv, d, page_size):
-        tile_req, tile_row0, n_tiles = ctx.attention_tiles(prefill_tokens)
+                                   rows, reqs, min_tiles=min_tiles, **options)
+    tile_req, tile_row0, n_tiles = ctx.attention_tiles(prefill_tokens, portions_only=tma_decode)
+    if n_tiles > 0:
         prefill_kernel(q, k_pages, v_pages, block_table, tile_req, tile_row0, n_tiles, ctx.q_start,
-                       ctx.positions, scale, window, out)
-    else:
-        tile_req, tile_row0, n_tiles = ctx.attention_tiles(MMA_KEYS // (nh // nkv))
-        paged_attention_mma(q, k_pages, v_pages, block_table, tile_req, tile_row0, n_tiles, ctx.q_start,
-                            ctx.positions, scale, window, out, False)
+                       ctx.positions, scale, window, out, **options)
 
 
 def joint_mma_attention_supported(dtype: torch.dtype, n_heads: int, n_kv_heads: int, head_dim: int, value_dim: int,

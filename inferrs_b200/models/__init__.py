@@ -5,3 +5,4 @@ from . import tikizen  # noqa: F401
 from . import sefalorn  # noqa: F401
 from . import ruzunex  # noqa: F401
 from . import dasusun  # noqa: F401
+from . import puposun  # noqa: F401

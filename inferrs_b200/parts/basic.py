@@ -15,8 +15,9 @@ from .spec import NormSpec, PositionSpec, TensorDecl
 def _nothing_pending(delta):
     """A block that norms after the sum hands on a copy of the stream instead of an output that is still to be
     added (an object with ``rows`` and no ``delta``): for a norm that means that nothing is pending.  A gated
-    output (:class:`GatedUpdate`) becomes plain rows here, for the norms that do not apply the gate themselves."""
-    if isinstance(delta, GatedUpdate):
+    output (:class:`GatedUpdate`) or one with a bias (:class:`SumUpdate`) becomes plain rows here, for the norms that do
+    not apply these themselves."""
+    if isinstance(delta, (GatedUpdate, SumUpdate)):
         return delta.rows()
     return None if (delta is not None and hasattr(delta, "rows") and not hasattr(delta, "delta")) else delta
 
@@ -56,6 +57,30 @@ class SandwichUpdate:
         self.source, self.average, self.result = source, average, result
 
 
+class SumUpdate:
+    """A pending output with what joins the residual stream beside it: x += delta + bias + plus.  ``bias`` (float32
+    [width]) belongs to the output, ``plus`` are float32 rows (an embedding that is added again).  The norm kernel that
+    follows does it (:class:`RMSNorm`)."""
+
+    def __init__(self, delta: Optional[torch.Tensor], bias: Optional[torch.Tensor] = None,
+                 plus: Optional[torch.Tensor] = None):
+        self.delta, self.bias, self.plus = delta, bias, plus
+
+    def rows(self) -> Optional[torch.Tensor]:
+        if self.plus is not None:
+            raise ValueError("float rows join the residual stream through an RMS norm without groups")
+        if self.bias is not None:
+            kernels.bias_add(self.delta, self.bias)
+        return self.delta
+
+    @staticmethod
+    def of(pending) -> Optional["SumUpdate"]:
+        """A pending output as a sum; None if it joins the stream in another way."""
+        if isinstance(pending, SumUpdate):
+            return pending
+        return SumUpdate(pending) if pending is None or isinstance(pending, torch.Tensor) else None
+
+
 class RMSNorm:
     """x / sqrt(mean(x^2) + eps) * w, in float32 (inferrs-kernels/candle-kernels/src/reduce.cu:188-228),
     fused with the residual addition that precedes it in a block.  With ``groups`` > 1 every one of that many equal
@@ -64,6 +89,7 @@ class RMSNorm:
     sum (``read``; None: the plain sum).  With a ``weight_offset`` the weight is offset + the stored one, in float32."""
 
     graph_safe = True  # launches depend only on shapes, never on the step's host-side values
+    routes_rows = True     # ``add_norm`` takes a ``router``
 
     @staticmethod
     def declare(spec: NormSpec) -> List[TensorDecl]:
@@ -81,9 +107,15 @@ class RMSNorm:
             self.weight = self.weight.to(torch.float32) + offset
 
     def add_norm(self, residual: torch.Tensor, delta, rows: Optional[torch.Tensor] = None,
-                 read: Optional[torch.Tensor] = None, conv=None):
+                 read: Optional[torch.Tensor] = None, conv=None, router=None):
         """``conv``: the arguments of the convolution that follows, for a step of single rows
-        (:func:`~inferrs_b200.kernels.sandwich_norm`)."""
+        (:func:`~inferrs_b200.kernels.sandwich_norm`).  ``router``: the experts' weights of the normed rows are made by
+        the same kernel, and (rows, weights) come back."""
+        if router is not None or isinstance(delta, SumUpdate):
+            if residual.dim() == 2 and getattr(self.spec, "groups", 1) == 1 and read is None and conv is None:
+                return self._sum(residual, delta, rows, router)
+            if router is not None:
+                raise ValueError("rows are routed behind a norm without groups on a residual of one stream")
         if isinstance(delta, SandwichUpdate) or conv is not None:
             return self._sandwich(residual, delta, rows, conv)
         delta = _nothing_pending(delta)
@@ -106,6 +138,17 @@ class RMSNorm:
         out = torch.empty((n, self.spec.size), dtype=self.rt.dtype, device=residual.device)
         kernels.add_rms_norm(residual, delta, self.weight, self.spec.eps, out, rows)
         return out
+
+    def _sum(self, residual: torch.Tensor, pending, rows: Optional[torch.Tensor], router):
+        u = SumUpdate.of(pending)
+        if u is None or residual.dim() != 2 or getattr(self.spec, "groups", 1) != 1:
+            raise ValueError("a sum of pending outputs joins the plain residual [rows, width] through a norm without groups")
+        n = residual.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((n, self.spec.size), dtype=self.rt.dtype, device=residual.device)
+        shares = None if router is None else torch.empty((n, router.columns), dtype=torch.float32, device=residual.device)
+        kernels.sum_norm_route(residual, u.delta, u.bias, u.plus if rows is None else None, self.weight, self.spec.eps, out,
+                               rows=rows, router=router, shares=shares)
+        return out if router is None else (out, shares)
 
     def _sandwich(self, residual: torch.Tensor, delta, rows: Optional[torch.Tensor], conv):
         u = delta if isinstance(delta, SandwichUpdate) else SandwichUpdate(_nothing_pending(delta))
@@ -268,6 +311,12 @@ class RotaryScaled:
         return self.cos, self.sin, self.spec.rot_dim
 
 
+class RotaryScaledInterleaved(RotaryScaled):
+    """The same tables; element 2i of a head is rotated with element 2i + 1."""
+
+    interleaved = True
+
+
 class NoPosition:
     def __init__(self, spec: PositionSpec, rt: Runtime):
         self.spec = spec
@@ -279,6 +328,7 @@ class NoPosition:
 register_position("rotary_split_half", RotarySplitHalf)
 register_position("rotary_interleaved", RotaryInterleaved)
 register_position("rotary_scaled", RotaryScaled)
+register_position("rotary_scaled_interleaved", RotaryScaledInterleaved)
 register_position("none", NoPosition)
 
 

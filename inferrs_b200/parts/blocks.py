@@ -7,7 +7,7 @@ import torch
 
 from .. import kernels
 from ..cache.storage import StateNeed
-from .basic import GatedUpdate, Linear, SandwichUpdate, StreamUpdate
+from .basic import GatedUpdate, Linear, SandwichUpdate, StreamUpdate, SumUpdate, fuse_rows
 from .registry import register_arrangement
 from .spec import TensorDecl
 
@@ -423,3 +423,94 @@ def depth_planes(spec) -> int:
 
 
 register_arrangement("sandwich", SandwichBlock)
+
+
+class ParallelBlock:
+    """h = norm(x), x += the sum of part(h) over all sub-layers: there is one norm, the first sub-layer's, and every
+    sub-layer reads its output.
+
+    Where all parts let their products be joined (``joins_products``), the block has two: one makes every part's
+    projections of h side by side, each part turns its columns into its columns of one wide row (``middle``), and the
+    second product takes that row to the sum of the parts' outputs, because [A | B] [a; b] = A a + B b; the addition of
+    the sub-layers is part of its float32 accumulation.  A part that routes rows (``router_beside_norm``) has its choice made
+    by the norm's kernel where that is better.  Parts that do not join run one after the other, and their outputs are
+    added.
+
+    As in :class:`SequentialBlock` nothing is added to the stream where the block ends: its output is handed on (with the
+    joined products' bias as a :class:`~inferrs_b200.parts.basic.SumUpdate`)."""
+
+    PAD_ROWS = 64        # the joined projection's rows are filled up to a multiple of this
+
+    def __init__(self, spec, sublayers: List[BuiltSubLayer]):
+        if not sublayers:
+            raise ValueError("a layer needs at least one sub-layer")
+        if isinstance(sublayers[0].norm, _no_norm()) or not hasattr(sublayers[0].norm, "add_norm") \
+                or any(not isinstance(s.norm, _no_norm()) for s in sublayers[1:]) \
+                or any(s.post_norm is not None or s.sum_norm is not None or s.part is None for s in sublayers):
+            raise ValueError("the sub-layers of a parallel block have one norm, before the first of them")
+        self.spec = spec
+        self.sublayers = list(sublayers)
+        self.norm = sublayers[0].norm
+        self.routed = [s.part for s in sublayers if hasattr(s.part, "router_beside_norm")]
+        self.joined = all(getattr(s.part, "joins_products", lambda: False)() for s in sublayers)
+        if self.joined:
+            self._join(self.norm.rt)
+
+    def _join(self, rt):
+        ins, outs, biases = zip(*[s.part.hand_over_products() for s in self.sublayers])
+        self.in_cols = _columns([w.shape[0] for w in ins])
+        self.mid_cols = _columns([w.shape[1] for w in outs])
+        n_in = self.in_cols[-1][1]
+        pad = -n_in % self.PAD_ROWS
+        fill = [torch.zeros((pad, ins[0].shape[1]), dtype=ins[0].dtype, device=ins[0].device)] if pad else []
+        self.in_product = Linear(fuse_rows(list(ins) + fill), rt)
+        if len({w.dtype for w in outs}) > 1:
+            outs = [w.to(torch.float32) for w in outs]
+        self.out_product = Linear(torch.cat(list(outs), dim=1).contiguous(), rt)
+        biases = [b.to(torch.float32) for b in biases if b is not None]
+        self.bias = sum(biases[1:], biases[0]).contiguous() if biases else None
+
+    def parts(self):
+        yield self.norm
+        for s in self.sublayers:
+            yield s.part
+
+    def forward(self, ctx, cache_id: int, residual: torch.Tensor, pending):
+        if residual.dim() != 2:
+            raise ValueError("a parallel block runs on the plain residual [rows, width]")
+        n = residual.shape[0]
+        router = self.routed[0].router_beside_norm(n) if len(self.routed) == 1 and self.joined \
+            and getattr(self.norm, "routes_rows", False) and SumUpdate.of(pending) is not None else None
+        shares = None
+        if router is not None:
+            h, shares = self.norm.add_norm(residual, pending, router=router)
+        else:
+            h = self.norm.add_norm(residual, pending)
+        if not self.joined:
+            total = None
+            for s in self.sublayers:
+                y = s.run_part(ctx, cache_id, h)
+                if total is None:
+                    total = y
+                else:
+                    before, total = total, torch.empty_like(y)
+                    kernels.scaled_sum(before, 1.0, y, 1.0, total)
+            return total
+        proj = self.in_product(h)
+        mid = torch.empty((n, self.mid_cols[-1][1]), dtype=proj.dtype, device=proj.device)
+        for s, (c0, c1), (m0, m1) in zip(self.sublayers, self.in_cols, self.mid_cols):
+            s.part.middle(ctx, cache_id, h, proj[:, c0:c1], mid[:, m0:m1], shares=shares if s.part in self.routed else None)
+        y = self.out_product(mid)
+        return y if self.bias is None else SumUpdate(y, self.bias)
+
+
+def _columns(sizes):
+    """(first, one past the last) of consecutive runs of these sizes."""
+    out, at = [], 0
+    for n in sizes:
+        out.append((at, at + n))
+        at += n
+    return out
+
+
+register_arrangement("parallel", ParallelBlock)

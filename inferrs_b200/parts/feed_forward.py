@@ -89,6 +89,9 @@ class Dense:
 register_feed_forward("dense", Dense)
 
 
+ROUTER_BESIDE_NORM_BYTES = 64 << 20     # what the rows' blocks may read of a router matrix from L2, all together
+
+
 class RoutedExperts:
     """A mixture of small gated feed-forwards (see :class:`~inferrs_b200.parts.spec.RoutedExpertsSpec`).
 
@@ -110,6 +113,8 @@ class RoutedExperts:
         d = [TensorDecl(spec.router, (len(spec.experts), spec.width))]
         if spec.router_bias is not None:
             d.append(TensorDecl(spec.router_bias, (len(spec.experts),), init="uniform:0:0.1"))
+        if spec.correction is not None:
+            d.append(TensorDecl(spec.correction, (len(spec.experts),), init="uniform:0:0.1"))
         for gate, up, down in spec.experts:
             d += [TensorDecl(gate, (spec.inner, spec.width)), TensorDecl(up, (spec.inner, spec.width)),
                   TensorDecl(down, (spec.width, spec.inner))]
@@ -152,7 +157,14 @@ class RoutedExperts:
             router.append(weights[spec.shared[3]].reshape(1, spec.width))
         self.total_inner = n * spec.inner + (spec.shared_inner if self.has_shared else 0)
         self.router = Linear(fuse_rows(router), rt)
-        self.router_bias = None if spec.router_bias is None else weights[spec.router_bias].to(torch.float32).contiguous()
+        if spec.groups and (n % spec.groups or not 0 < spec.groups_keep <= spec.groups
+                            or spec.groups_keep * (n // spec.groups) < spec.top):
+            raise ValueError(f"routed experts: {spec.groups_keep} of {spec.groups} groups of {n} experts do not hold the "
+                             f"{spec.top} that are chosen")
+        f32 = lambda name: None if name is None else weights[name].to(torch.float32).contiguous()     # noqa: E731
+        self.routing = kernels.Router(n_experts=n, top=spec.top, bias=f32(spec.router_bias), correction=f32(spec.correction),
+                                      has_shared=self.has_shared, groups=spec.groups, keep=spec.groups_keep, mode=self.mode,
+                                      scale=float(spec.route_scale), weight=self.router.weight)
         self.gate_up = Linear(fuse_rows(gates + ups), rt)
         if len({t.dtype for t in downs}) > 1:
             downs = [t.to(torch.float32) for t in downs]
@@ -160,14 +172,33 @@ class RoutedExperts:
 
     def forward(self, ctx, h):
         n = h.shape[0]
-        logits = self.router(h, out_dtype=torch.float32)
-        share = torch.empty((n, self.n_experts + int(self.has_shared)), dtype=torch.float32, device=h.device)
-        kernels.router_topk(logits, self.router_bias, self.n_experts, self.spec.top, self.has_shared, share,
-                            self.rt.dtype, mode=self.mode, scale=self.spec.route_scale)
         a = torch.empty((n, self.total_inner), dtype=self.rt.dtype, device=h.device)
-        kernels.routed_gate(self.gate_up(h), share, self.n_experts, self.spec.inner, a, limit=self.limit,
-                            slope=self.spec.slope)
+        self.middle(ctx, None, h, self.gate_up(h), a)
         return self.down(a)
+
+    # A block whose sub-layers all read the same rows may make this part's products in one with the others', and let
+    # the norm's kernel choose the experts (see ParallelBlock).
+    def joins_products(self) -> bool:
+        return self.gate_up is not None
+
+    def hand_over_products(self):
+        products = (self.gate_up.weight, self.down.weight, None)
+        self.gate_up = self.down = None
+        return products
+
+    def router_beside_norm(self, n_rows: int):
+        """The router for a norm kernel that makes its logits too; None where a product of its own is better (many
+        rows: every row's block reads the whole matrix)."""
+        w = self.router.weight
+        fits = n_rows * w.numel() * w.element_size() <= ROUTER_BESIDE_NORM_BYTES
+        return self.routing if fits and kernels.sum_norm_routes(self.spec.width, self.routing) else None
+
+    def middle(self, ctx, cache_id, h, proj: torch.Tensor, out: torch.Tensor, shares=None):
+        """The experts' inner rows times their weights (``shares``: the weights, if they are made already)."""
+        if shares is None:
+            shares = torch.empty((h.shape[0], self.routing.columns), dtype=torch.float32, device=h.device)
+            kernels.route(self.router(h, out_dtype=torch.float32), self.routing, shares, self.rt.dtype)
+        kernels.routed_gate(proj, shares, self.n_experts, self.spec.inner, out, limit=self.limit, slope=self.spec.slope)
 
 
 register_feed_forward("routed_experts", RoutedExperts)

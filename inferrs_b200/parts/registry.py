@@ -40,6 +40,13 @@ of ``forward``.  A part that has them may be handed :class:`~inferrs_b200.kernel
 output, and a :class:`~inferrs_b200.kernels.ResidualSink` in place of returning its result (see
 :class:`~inferrs_b200.parts.blocks.SequentialBlock`); a part without them never sees either.
 
+Optional for mixers and feed-forwards: ``joins_products() -> bool``, ``hand_over_products() -> (in [n, width],
+out [width, m], bias of the output or None)`` (the part gives up its own copies) and ``middle(ctx, cache_id, h, proj, out,
+shares=None)``: from its n columns of a wider projection of h to its m columns of a wider row.  With them a block whose
+sub-layers all read the same rows makes their products in one (see :class:`~inferrs_b200.parts.blocks.ParallelBlock`).
+``router_beside_norm(n_rows) -> Router | None``: the routing that the norm's kernel may do for the part; ``shares`` are its
+results.
+
 Every part may set ``graph_safe = True`` to say that its launches depend only on shapes and device
 memory, never on host-side values of the step; a model whose parts all say so has its steps captured
 into CUDA graphs.  A part without the attribute keeps the model's steps launched one by one.

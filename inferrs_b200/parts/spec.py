@@ -58,6 +58,8 @@ class PositionSpec:
     turns(t) = rot_dim ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(turns(fast)), 0),
     hi = min(ceil(turns(slow)), rot_dim - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), pair i turns at
     f_i / factor * ramp_i + f_i (1 - ramp_i), and cos and sin are multiplied by 0.1 ln(factor) + 1).
+    ``kind="rotary_scaled_interleaved"`` does the same with the pairs ``2i``, ``2i + 1``.  (The two scaled kinds make
+    their angles in float64, with and without a stretch.)
     """
 
     kind: str = "rotary_split_half"
@@ -92,6 +94,13 @@ class AttentionSpec:
     ``norm_whole``: ``q_norm`` / ``k_norm`` are taken over the whole projection, all heads at once (their ``size`` is
     n_heads * head_dim and n_kv_heads * head_dim), instead of per head.
     ``gate_proj`` [n_heads * value_dim, width]: the heads side by side are multiplied by sigmoid(gate(x)) before
+    ``o_proj``.
+    ``value_is_key``: there is no ``v_proj``; a value is its key as it was projected (with ``k_bias``, before norm and
+    rotation).
+    ``score_cap``: after scale, factor and distance terms a score becomes cap * tanh(score / cap).
+    ``sink_score``: like ``sink`` with one constant score for all heads.
+    ``keep_first``: beside its ``window`` a query also sees the sequence's first keys, j < keep_first (and j <= i).
+    ``head_gate`` [n_heads, width]: head h's output is multiplied by sigmoid((head_gate x)_h), one number per head, before
     ``o_proj``.
     ``value_publish``: the layer's values of the step's rows, as they are cached, are kept under this name for later
     layers of the same step.  ``value_blend`` = (name, weight tensor of one number): v <- (1 - w) v + w v_name with
@@ -133,6 +142,11 @@ class AttentionSpec:
     value_publish: Optional[str] = None
     value_blend: Optional[Tuple[str, str]] = None
     unused: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()
+    value_is_key: bool = False
+    score_cap: Optional[float] = None
+    sink_score: Optional[float] = None
+    keep_first: int = 0
+    head_gate: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -175,6 +189,9 @@ class RoutedExpertsSpec:
     ``scoring="sigmoid_share"``: the scores are s = sigmoid(z), the ``top`` largest scores are chosen, and a chosen
     expert weighs s_e / (sum of the chosen scores + 1e-20).  ``scoring="softmax_share"``: the same with the scores
     s = softmax(z) over all experts.  ``route_scale`` multiplies the routed experts' weights.
+    ``correction`` [experts]: experts are chosen by score + correction; the weights use the score without it.
+    ``groups`` > 0: the experts form that many equal groups of neighbours, a group's worth is the sum of its two largest
+    choice scores, and only the experts of the ``groups_keep`` best groups can be chosen.
     ``activation="clamped_swish"`` (with ``limit`` and ``slope``): an expert is down_e( g sigmoid(slope g) (u + 1) )
     with g = min(gate_e(x), limit) and u = clamp(up_e(x), -limit, limit)."""
 
@@ -192,6 +209,9 @@ class RoutedExpertsSpec:
     activation: str = "silu"
     limit: Optional[float] = None
     slope: float = 1.702
+    correction: Optional[str] = None
+    groups: int = 0
+    groups_keep: int = 0
 
 
 @dataclass(frozen=True)
@@ -521,6 +541,8 @@ class LayerSpec:
     ``input_conv``, x += layer_scale * post_norm(part(h)); and where the layer has a ``depth_average``, what it hands on
     is that average of the results so far.
 
+    ``arrangement="parallel"``: h = norm(x) with the first sub-layer's norm, x += the sum of part(h) over all sub-layers.
+
     ``unused``: tensors that the weight files hold for this layer and that nothing reads, as (name, shape).
     """
 
@@ -570,10 +592,13 @@ class ScheduleEntry:
     ``cache`` numbers the caches (and fixed-size states) of the model.  Two
     entries with the same ``layer`` share weights; two entries with the same
     ``cache`` share keys and values (exactly one of them writes).
+    ``add_embedding``: the embedding output (as it enters the first layer) is added to the residual stream before the
+    layer runs.
     """
 
     layer: int
     cache: int
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)
@@ -603,6 +628,17 @@ class ModelSpec:
     eos_token_ids: Tuple[int, ...] = ()
     architecture: str = ""
     extra: Tuple[Tuple[str, Any], ...] = field(default_factory=tuple)
+
+
+def looped_schedule(n_layers: int, start: int, stop: int, times: int, add_embedding: bool = False
+                    ) -> Tuple[ScheduleEntry, ...]:
+    """Layers start .. stop - 1 run ``times`` times in a row, the others once; every run has a cache of its own.
+    ``add_embedding``: the embedding output joins the stream at the start of every pass but the first."""
+    order = [(i, False) for i in range(start)]
+    for t in range(times):
+        order += [(i, add_embedding and t > 0 and i == start) for i in range(start, stop)]
+    order += [(i, False) for i in range(stop, n_layers)]
+    return tuple(ScheduleEntry(layer=i, cache=k, add_embedding=again) for k, (i, again) in enumerate(order))
 
 
 def default_schedule(n_layers: int) -> Tuple[ScheduleEntry, ...]:

@@ -13,8 +13,10 @@ from typing import Optional
 import torch
 
 
-def embedding_gather(table, ids, out, act_dtype=None, scale=1.0):
+def embedding_gather(table, ids, out, act_dtype=None, scale=1.0, copy=None):
     out.copy_(table[ids.long()].float() * scale)
+    if copy is not None:
+        copy.copy_(out)
 
 
 def rms_norm_rows(x, weight, eps, out):
@@ -78,13 +80,13 @@ def _rotate(x, cos, sin, rot_dim, interleaved=False):
 
 def qk_norm_rope_store(qkv, n_heads, n_kv_heads, head_dim, store_kv, q_weight, k_weight, eps, cos, sin, rot_dim,
                        positions, row_request, block_table, k_pages, v_pages, q_out, interleaved=False, norm_q=None,
-                       norm_k=None, norm_after_rotation=False):
+                       norm_k=None, norm_after_rotation=False, bias=None, value_is_key=False):
     # the plain order only (norm, then rotation; a normed kind has its weight; values as large as keys)
     assert not norm_after_rotation and norm_q in (None, q_weight is not None) and \
         norm_k in (None, k_weight is not None and store_kv, k_weight is not None)
     n = qkv.shape[0]
     d = head_dim
-    x = qkv.float()
+    x = qkv.float() if bias is None else qkv[:, :bias.shape[0]].float() + bias
     q = x[:, :n_heads * d].reshape(n, n_heads, d)
     pos = positions.long()
     if q_weight is not None:
@@ -95,7 +97,8 @@ def qk_norm_rope_store(qkv, n_heads, n_kv_heads, head_dim, store_kv, q_weight, k
     if not store_kv:
         return
     k = x[:, n_heads * d:(n_heads + n_kv_heads) * d].reshape(n, n_kv_heads, d)
-    v = x[:, (n_heads + n_kv_heads) * d:].reshape(n, n_kv_heads, d)
+    first = n_heads if value_is_key else n_heads + n_kv_heads
+    v = x[:, first * d:(first + n_kv_heads) * d].reshape(n, n_kv_heads, d)
     if k_weight is not None:
         k = _rms(k, k_weight, eps)
     if rot_dim:
@@ -113,7 +116,8 @@ def qk_norm_rope_store(qkv, n_heads, n_kv_heads, head_dim, store_kv, q_weight, k
             v_pages[page, :, p % page_size + 1:, :] = 0
 
 
-def paged_attention_generic(q, k_pages, v_pages, block_table, row_request, positions, scale, window, out):
+def paged_attention_generic(q, k_pages, v_pages, block_table, row_request, positions, scale, window, out, head_scale=None,
+                            slopes=None, sinks=None, cap=None, keep_first=0, gate=None):
     n, nh, d = q.shape
     nkv, page_size = k_pages.shape[1], k_pages.shape[2]
     g = nh // nkv
@@ -121,7 +125,8 @@ def paged_attention_generic(q, k_pages, v_pages, block_table, row_request, posit
         pos = int(positions[r])
         req = int(row_request[r])
         lo = (max(0, pos - window + 1) if window > 0 else (pos // -window) * -window) if window else 0
-        js = torch.arange(lo, pos + 1)
+        js = torch.arange(0, pos + 1)
+        js = js[(js >= lo) | (js < keep_first)].to(k_pages.device)
         pages = block_table[req, (js // page_size).long()].long()
         assert (pages >= 0).all(), "a visible key lies in a page that was given back"
         k = k_pages[pages, :, (js % page_size).long(), :].float()  # [keys, nkv, d]
@@ -129,13 +134,83 @@ def paged_attention_generic(q, k_pages, v_pages, block_table, row_request, posit
         k = k.repeat_interleave(g, dim=1)
         v = v.repeat_interleave(g, dim=1)
         s = torch.einsum("hd,khd->hk", q[r].float(), k) * scale
-        p = torch.softmax(s, dim=-1)
+        if head_scale is not None:
+            s = s * head_scale[:, None]
+        if slopes is not None:
+            s = s - slopes[:, None] * (pos - js)[None, :]
+        if cap is not None:
+            s = cap * torch.tanh(s / cap)
+        if sinks is not None:
+            p = torch.softmax(torch.cat([s, sinks[:, None]], dim=-1), dim=-1)[:, :-1]
+        else:
+            p = torch.softmax(s, dim=-1)
         o = torch.einsum("hk,khd->hd", p, v)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[r, :nh].float())[:, None]
         out[r] = o.reshape(nh * d).to(out.dtype)
 
 
-def paged_attention(q, k_pages, v_pages, block_table, ctx, scale, window, out):
-    paged_attention_generic(q, k_pages, v_pages, block_table, ctx.row_request, ctx.positions, scale, window, out)
+def paged_attention(q, k_pages, v_pages, block_table, ctx, scale, window, out, **options):
+    paged_attention_generic(q, k_pages, v_pages, block_table, ctx.row_request, ctx.positions, scale, window, out, **options)
+
+
+def bias_add(x, bias):
+    x[:, :bias.shape[0]] = (x[:, :bias.shape[0]].float() + bias).to(x.dtype)
+
+
+def scaled_sum(x, a, y, b, out):
+    out.copy_((a * x.float() + b * y.float()).to(out.dtype))
+
+
+def route(logits, router, weights, act_dtype=None):
+    """Row by row: scores, the best groups, the chosen experts, their weights (csrc/router.cuh)."""
+    n = router.n_experts
+    for r in range(logits.shape[0]):
+        z = logits[r, :n].double()
+        if router.bias is not None:
+            z = z + router.bias.double()
+        s = {0: z, 1: torch.sigmoid(z), 2: torch.softmax(z, dim=-1)}[router.mode].tolist()
+        c = [a + (float(router.correction[e]) if router.correction is not None else 0.0) for e, a in enumerate(s)]
+        allowed = list(range(n))
+        if router.groups:
+            size = n // router.groups
+            worth = [sum(sorted(c[g * size:(g + 1) * size])[-2:]) for g in range(router.groups)]
+            best = sorted(range(router.groups), key=lambda g: -worth[g])[:router.keep]
+            allowed = sorted(e for g in best for e in range(g * size, (g + 1) * size))
+        chosen = sorted(allowed, key=lambda e: -c[e])[:router.top]
+        share = torch.softmax(torch.tensor([s[e] for e in chosen]), dim=0).tolist() if router.mode == 0 \
+            else [s[e] / (sum(s[k] for k in chosen) + 1e-20) for e in chosen]
+        weights[r] = 0.0
+        for e, w in zip(chosen, share):
+            weights[r, e] = w * router.scale
+        if router.has_shared:
+            weights[r, n] = torch.sigmoid(logits[r, n])
+
+
+def routed_gate(gate_up, weights, n_experts, ff, out, limit=None, slope=1.702):
+    inner = out.shape[1]
+    g, u = gate_up[:, :inner].float(), gate_up[:, inner:].float()
+    if limit is None:
+        a = g * torch.sigmoid(g) * u
+    else:
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        a = g * torch.sigmoid(slope * g) * (u + 1.0)
+    col = (torch.arange(inner, device=out.device) // ff).clamp(max=weights.shape[1] - 1)
+    out.copy_((a * weights[:, col]).to(out.dtype))
+
+
+def sum_norm_route(residual, delta, bias, plus, weight, eps, out, rows=None, router=None, shares=None):
+    x = residual
+    for t in (delta, bias, plus):
+        if t is not None:
+            x = x + t.float()
+    if rows is None:
+        residual.copy_(x)
+    else:
+        x = x[rows.long()]
+    out.copy_((x / torch.sqrt((x * x).mean(dim=-1, keepdim=True) + eps) * weight.float()).to(out.dtype))
+    if router is not None:
+        route(out.float() @ router.weight.float().t(), router, shares)
 
 
 def gemm_tn_simt(x, w, out, act_dtype=None):
@@ -233,4 +308,5 @@ def sample(logits, temperature, top_k, top_p, min_p, uniform, out, act_dtype=Non
         out[r] = int(order[int(hit[0])]) if len(hit) else int(order[-1])
 
 
-_NAMES += ["penalties", "sample", "rms_norm_rows", "add_cast", "logit_scale_softcap"]
+_NAMES += ["penalties", "sample", "rms_norm_rows", "add_cast", "logit_scale_softcap", "bias_add", "scaled_sum", "route",
+           "routed_gate", "sum_norm_route"]

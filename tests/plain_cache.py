@@ -65,6 +65,7 @@ class GroupLayout:
 
     name: str
     window: Optional[int] = None  # None: all keys; w: a query at i sees keys j with i - w < j <= i
+    keep_first: int = 0           # beside its window a query also sees keys j < keep_first
 
 
 @dataclass
@@ -192,10 +193,11 @@ class CacheManager:
             if first_needed <= 0:
                 continue
             dead = first_needed // self.page_size  # pages 0..dead-1 hold only keys < first_needed
-            gone = [p for p in r.tables[g][:dead] if p != RELEASED]
+            first = self._pages_for(layout.keep_first)      # the pages of the sequence's first keys stay
+            gone = [p for p in r.tables[g][first:dead] if p != RELEASED]
             if gone:
                 self.pools[g].give_back(gone)
-                for i in range(dead):
+                for i in range(first, dead):
                     r.tables[g][i] = RELEASED
 
     def release(self, rid: Hashable):

@@ -87,6 +87,26 @@ def test_window_group_gives_pages_back_when_the_window_has_passed():
     assert m.pools[0].n_free == 16 and m.pools[1].n_free == 16
 
 
+def test_pages_of_the_first_tokens_stay_when_the_window_has_passed_them():
+    """A window of 6 beside the first 5 tokens, pages of 4: the pages 0 and 1 (tokens 0..7) stay for good, every other
+    page goes back as soon as the window has passed its last token; all of them are free after the request's end."""
+    m = CacheManager([GroupLayout("win", window=6, keep_first=5)], page_size=4, n_pages=[16], max_requests=2)
+    m.admit("r")
+    for n in range(1, 41):
+        m.reserve({"r": 1}); m.commit("r", 1)
+        table = m.block_table("r", 0)
+        first_needed = n - 6 + 1
+        for page, pid in enumerate(table):
+            gone = page >= 2 and (page + 1) * 4 <= first_needed
+            assert (pid == RELEASED) == gone, (n, page)
+        m.check_invariants()
+    assert m.pools[0].n_free == 16 - 4       # two kept, and the two that the window reaches into
+    m.release("r")
+    assert m.pools[0].n_free == 16
+    with pytest.raises(CacheError, match="keep_first"):
+        CacheManager([GroupLayout("win", window=6, keep_first=-1)], page_size=4, n_pages=[16], max_requests=2)
+
+
 @pytest.mark.parametrize("seed", range(6))
 def test_random_orders_never_lose_a_page(seed):
     rng = random.Random(seed)
@@ -126,9 +146,11 @@ def test_native_manager_answers_as_the_plain_model_does(seed):
     windows = [None, rng.choice([2, 5, 9, 33])] if seed % 2 else [rng.choice([4, 17]), None, None]
     page_size = rng.choice([1, 3, 16])
     n_pages = [rng.randint(5, 30) for _ in windows]
-    nat = CacheManager([GroupLayout(f"g{i}", w) for i, w in enumerate(windows)], page_size, n_pages, max_requests=5)
-    ref = plain_cache.CacheManager([plain_cache.GroupLayout(f"g{i}", w) for i, w in enumerate(windows)], page_size,
-                                   n_pages, max_requests=5)
+    keeps = [0 if w is None else rng.choice([0, 1, 5, 16, 40]) for w in windows]
+    nat = CacheManager([GroupLayout(f"g{i}", w, k) for i, (w, k) in enumerate(zip(windows, keeps))], page_size, n_pages,
+                       max_requests=5)
+    ref = plain_cache.CacheManager([plain_cache.GroupLayout(f"g{i}", w, k) for i, (w, k) in enumerate(zip(windows, keeps))],
+                                   page_size, n_pages, max_requests=5)
     live, next_id = [], 0
     for _ in range(500):
         op = rng.random()
