@@ -43,6 +43,14 @@ sides of every sub-layer, averages over depth, a short convolution in front of e
 latent attention in every layer, the closest existing model, at equal width, heads, latents, layers and feed-forward
 size, and the design's own kernels each beside the like kernel of the closest model.
 
+    python bench.py --design puposun [--design-layers N]
+
+does the same for the Puposun design (sub-layers side by side behind one norm with joined products, attention whose values
+are its keys: with a cap and a sink, or with a window beside the first tokens and a gate per head; routed experts chosen
+inside the best groups; also with its layers passed twice) beside the Ruzunex design with attention layers and routed
+experts alone, the closest existing model, and beside the Qwen3 shape, both at equal width, heads, layers and
+feed-forward size, and the design's own kernels each beside the like kernel of the closest model.
+
     python bench.py --design sefalorn [--design-layers N]
 
 does the same for the Sefalorn design (window attention with mixed heads and a distance penalty beside the gated
@@ -302,6 +310,43 @@ def dasusun_config(width: int, heads: int, ff: int, q_rank: int, kv_rank: int, n
             "canon": {"taps": 3}, "layers": [layer(i) for i in range(n_layers)]}
 
 
+def puposun_config(width: int, heads: int, ff: int, n_layers: int, vocab: int, passes: int = 1) -> dict:
+    """A window of 1,024 beside the first four tokens in three of four layers, every earlier key in the fourth; eight
+    experts of ff / 8 in four groups, two chosen.  ``passes`` > 1: n_layers / passes layers that run that many times."""
+    mlp = {"kind": "moe", "expert": {"ff": ff // 8},
+           "router": {"experts": 8, "top": 2, "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+    sizes = {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+             "rot": {"base": 1e6, "dims": 128}}
+
+    def layer(i):
+        if i % 4 == 3:
+            return {"type": "attention", "mlp": mlp, "mixer": dict(sizes, softcap=20.0)}
+        return {"type": "attention_2", "mlp": mlp, "mixer": dict(sizes, mask={"size": 1024, "keep_first": 4})}
+    own = max(n_layers // passes, 1)
+    return {"architecture": "Puposun", "vocab": vocab, "width": width, "max_positions": 8192, "norm": {"eps": 1e-5},
+            "embedding": {"scale": 1.0}, "logit_softcap": 15.0, "layers": [layer(i) for i in range(own)],
+            "loop": {"start": 0, "stop": own, "times": passes}}
+
+
+def ruzunex_attention_config(width: int, heads: int, ff: int, n_layers: int, vocab: int) -> dict:
+    """Ruzunex with attention layers alone (a window of 1,024 in three of four) and routed experts behind each."""
+    base = ruzunex_config(width, heads, ff, 2, vocab)
+    moe = base["layers"][1]["mlp"]
+
+    def layer(i):
+        m = dict(base["layers"][0]["mixer"])
+        if i % 4 == 3:
+            m.pop("mask")
+        return {"type": "attention", "mlp": moe, "mixer": m}
+    return dict(base, layers=[layer(i) for i in range(n_layers)])
+
+
+def qwen3_equal_config(width: int, heads: int, ff: int, n_layers: int, vocab: int) -> dict:
+    return dict(CONFIG_8B, num_hidden_layers=n_layers, hidden_size=width, num_attention_heads=heads,
+                num_key_value_heads=heads // 4, head_dim=128, intermediate_size=ff, vocab_size=vocab,
+                max_position_embeddings=8192)
+
+
 def vebonex_latent_config(width: int, heads: int, ff: int, q_rank: int, kv_rank: int, n_layers: int, vocab: int,
                           positions: int) -> dict:
     """Vebonex with latent attention (latents of its own) in every layer."""
@@ -383,6 +428,46 @@ def design_bench(args) -> int:
         r["frac_bf16"] = round(r["TFLOPs"] / pk["bf16_tflops"], 4)
         return r
 
+    if args.design == "puposun":
+        sizes = []
+        for name, width, heads, ff in (("width 2048", 2048, 16, 8192), ("width 4096", 4096, 32, 16384)):
+            size = (width, heads, ff, args.design_layers, vocab)
+            sizes.append({"size": name, "layers": args.design_layers, "heads": heads, "ff": ff,
+                          "puposun": measure(puposun_config(*size)),
+                          "puposun_half_the_layers_twice": measure(puposun_config(*size, passes=2)),
+                          "ruzunex_equal_size": measure(ruzunex_attention_config(*size)),
+                          "qwen3_equal_size": measure(qwen3_equal_config(*size))})
+        rows = []
+        for heads in (16, 32):
+            att = dict(context_before=0, splits=0, min_tiles=0, max_context=0, head_dim=128, heads=heads, kv_heads=heads // 4)
+            plain, like = dict(per_head=False, options="", keep=0), dict(per_head=True, options="", keep=0)
+            capped = dict(per_head=False, options="cap,sink", keep=0)
+            kept = dict(per_head=False, options="gate", keep=4)
+            for form, n, impls in (("prefill", 1, ("tcgen05", "tcgen05-pair")), ("decode", 8, ("tcgen05", "mma")),
+                                   ("decode", 64, ("tcgen05", "mma"))):
+                at = dict(form=form, batch=n, context=2048, tokens=2048, **att)
+                # every earlier key with a cap and a sink; the like kernel (a factor, a slope and a sink per head); plain
+                rows.append(microbench.attention(ns(impl="tcgen05", window=0, **at, **capped)))
+                rows.append(microbench.attention(ns(impl="tcgen05" if form == "prefill" else "mma", window=0, **at, **like)))
+                rows.append(microbench.attention(ns(impl=impls[1], window=0, **at, **plain)))
+                # the window beside the first tokens with a gate; the like kernel; the same kernel without kept keys and gate
+                for impl in (impls if form == "prefill" else impls[:1]):
+                    rows.append(microbench.attention(ns(impl=impl, window=1024, **at, **kept)))
+                rows.append(microbench.attention(ns(impl="tcgen05" if form == "prefill" else "mma", window=1024, **at, **like)))
+                rows.append(microbench.attention(ns(impl=impls[1], window=1024, **at, **plain)))
+            for form, n in (("prefill", 2048), ("decode", 8)):
+                for impl in ("shared", "shared-interleaved", "plain"):
+                    rows.append(microbench.store(ns(form=form, impl=impl, batch=n, context=2048, tokens=n, taps=0,
+                                                    heads=heads, kv_heads=heads // 4, head_dim=128)))
+        for n in (2048, 8):
+            for width in (2048, 4096):
+                for impl, experts in (("add", 0), ("sum", 0), ("streams", 0), ("route", 8), ("add-route", 8), ("route", 64),
+                                      ("add-route", 64)):
+                    rows.append(microbench.residual(ns(impl=impl, tokens=n, width=width, planes=0, taps=0, experts=experts)))
+        print(json.dumps({"design": "Puposun", "dtype": "bf16", "data": "synthetic: seeded uniform token ids, random weights",
+                          "prompt_len": PROMPT_LEN, "decode_batch": batch, "decode_steps": args.design_steps,
+                          "peaks": pk, "sizes": sizes, "kernels": [fractions(r) for r in rows]}))
+        return 0
     if args.design == "dasusun":
         sizes = []
         shapes = (("width 2048", 2048, 16, 8192, 768, 512), ("width 4096", 4096, 32, 16384, 1536, 512),
@@ -574,7 +659,7 @@ def main() -> int:
     ap.add_argument("--clock-interval-ms", type=int, default=200, help="how often nvidia-smi is asked for the clocks")
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 and 64 points and the prefill")
     ap.add_argument("--no-workloads", action="store_true", help="skip the Qwen3-0.6B and Qwen3-32B workloads")
-    ap.add_argument("--design", choices=["vebonex", "tikizen", "sefalorn", "ruzunex", "dasusun"],
+    ap.add_argument("--design", choices=["vebonex", "tikizen", "sefalorn", "ruzunex", "dasusun", "puposun"],
                     help="another workload: this design beside the closest model")
     ap.add_argument("--design-layers", type=int, default=8, help="layers of both models of --design")
     ap.add_argument("--design-steps", type=int, default=64, help="timed decode steps of --design")

@@ -481,6 +481,7 @@ IB_EXPORT int ib_paged_attention_decode_noalloc(const void* q, const void* k_pag
     if (n_rows <= 0 || n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads || head_dim <= 0 || page_size <= 0 ||
         max_pages <= 0 || n_splits <= 0)
         return IB_NOALLOC_ERR_ARGUMENT;
+    if (head_dim != 64 && head_dim != 128 && head_dim != 256) return IB_NOALLOC_ERR_UNSUPPORTED;
     const long long need = (long long)n_rows * n_heads * n_splits * (head_dim + 2);
     if (need > (long long)IB_NOALLOC_SCRATCH_FLOATS) return IB_NOALLOC_ERR_TOO_LARGE;
     float* scratch = nullptr;
@@ -504,7 +505,7 @@ IB_EXPORT const char* ib_paged_attention_decode_noalloc_strerror(int code) {
     switch (code) {
         case 0: return "success";
         case IB_NOALLOC_ERR_UNSUPPORTED:
-            return "sizes not taken: head_dim must be 32, 64, 80, 96, 128, 192 or 256, the page size must divide 64, and at most 16 "
+            return "sizes not taken: head_dim must be 64, 128 or 256, the page size must divide 64, and at most 16 "
                    "query heads may share a key/value head";
         case IB_NOALLOC_ERR_ARGUMENT: return "a size is zero or negative, or heads are not a multiple of kv heads";
         case IB_NOALLOC_ERR_TOO_LARGE:

@@ -26,7 +26,7 @@ extern "C" {
 #define IB_NOALLOC_SCRATCH_FLOATS (4 * 1024 * 1024)
 
 // Return codes: 0 success; > 0 a cudaError_t; the negative ones below.
-#define IB_NOALLOC_ERR_UNSUPPORTED (-1)  // head_dim not 32/64/80/96/128/192/256, page size does not divide 64, > 16 heads per kv head
+#define IB_NOALLOC_ERR_UNSUPPORTED (-1)  // head_dim not 64/128/256, page size does not divide 64, > 16 heads per kv head
 #define IB_NOALLOC_ERR_ARGUMENT (-2)     // a size is zero or negative, or heads are not a multiple of kv heads
 #define IB_NOALLOC_ERR_TOO_LARGE (-3)    // the call needs more scratch than IB_NOALLOC_SCRATCH_FLOATS
 #define IB_NOALLOC_ERR_BUILD (-4)        // the library was built without the bfloat16 kernels

@@ -104,22 +104,35 @@ def attention(args) -> dict:
     window = getattr(args, "window", 0) or None
     per_head = {}
     if getattr(args, "per_head", False):       # a factor, a slope and a sink per head
-        if args.impl not in ("mma", "tcgen05") or (args.impl == "tcgen05" and args.form == "decode"):
-            raise SystemExit("--per-head is an option of --impl mma and of the prefill form of --impl tcgen05")
         per_head = {"head_scale": 1.0 + 0.1 * torch.randn(nh, device=dev),
                     "slopes": torch.tensor([2.0 ** (-8.0 * (h + 1) / nh) for h in range(nh)], device=dev),
                     "sinks": torch.randn(nh, device=dev)}
-    seen = lambda n_keys: min(n_keys, window) if window else n_keys      # noqa: E731
+    named = [o for o in (getattr(args, "options", "") or "").split(",") if o]
+    keep = getattr(args, "keep", 0)
+    if set(named) - {"cap", "sink", "gate"}:
+        raise SystemExit("--options are cap, sink and gate, with commas between them")
+    if "cap" in named:
+        per_head["cap"] = 20.0
+    if "sink" in named:
+        per_head["sinks"] = torch.zeros(nh, device=dev)
+    if "gate" in named:
+        per_head["gate"] = torch.randn(n, nh, device=dev).to(torch.bfloat16)
+    if keep:
+        per_head["keep_first"] = keep
+    if args.impl == "tcgen05-pair" and set(per_head) - {"gate", "keep_first"}:
+        raise SystemExit("--impl tcgen05-pair takes kept keys and the gate only")
+    seen = lambda n_keys: min(n_keys, window + keep) if window else n_keys      # noqa: E731
     if args.form == "decode":
         if args.impl == "mma":
             splits = args.splits or kernels.decode_splits(args.batch, nkv, seen(args.context))
             fn = lambda: kernels.paged_attention_mma(q, k_pages, v_pages, table, row_request, q_start, n, q_start,  # noqa: E731
                                                      positions, scale, window, out, True, splits, **per_head)
         else:
-            splits, min_tiles = kernels.decode_slices(args.batch, nkv, args.max_context or args.context)
+            reach = seen(args.context) + 2 * kernels.MMA_KEYS if window else args.context
+            splits, min_tiles = kernels.decode_slices(args.batch, nkv, args.max_context or min(reach, args.context))
             splits, min_tiles = args.splits or splits, args.min_tiles or min_tiles
             fn = lambda: kernels.paged_attention_decode(q, k_pages, v_pages, table, positions, scale, window, out,  # noqa: E731
-                                                        splits, min_tiles=min_tiles)
+                                                        splits, min_tiles=min_tiles, **per_head)
         byts = 2 * 2 * sum(seen(n_keys) for n_keys in lens) * nkv * d
         flops = 4 * nh * d * sum(seen(n_keys) for n_keys in lens)
         extra = {"batch": args.batch, "context": args.context, "splits": splits}
@@ -135,7 +148,7 @@ def attention(args) -> dict:
                                                          q_start, positions, scale, window, out, **per_head)
         elif args.impl == "tcgen05-pair":
             fn = lambda: kernels.paged_attention_pair_tcgen05(q, k_pages, v_pages, table, tile_req, tile_row0, len(req),  # noqa: E731
-                                                              q_start, positions, scale, window, out)
+                                                              q_start, positions, scale, window, out, **per_head)
         else:
             fn = lambda: kernels.paged_attention_mma(q, k_pages, v_pages, table, tile_req, tile_row0, len(req),  # noqa: E731
                                                      q_start, positions, scale, window, out, False, **per_head)
@@ -145,8 +158,10 @@ def attention(args) -> dict:
         extra = {"tokens": args.tokens, "context_before": args.context_before}
     if window:
         extra["window"] = window
-    if per_head:
+    if getattr(args, "per_head", False):
         extra["per_head"] = "factor, slope, sink"
+    if named or keep:
+        extra["options"] = ", ".join(named + ([f"first {keep} keys"] if keep else []))
     us = _time(fn, args.iters)
     return dict({"kernel": f"attention/{args.form}" + (f"/{args.impl}" if args.form == "prefill" else ""), "heads": nh, "kv_heads": nkv, "head_dim": d, "us": round(us, 2),
                  "GBps": round(byts / us / 1e3, 1), "TFLOPs": round(flops / us / 1e6, 1)}, **extra)
@@ -191,7 +206,8 @@ def scan(args) -> dict:
 
 def store(args) -> dict:
     """What stands between the q | k | v projection and the attention kernel, alone: the kernel that norms per head,
-    turns and stores (``--impl plain``), or the one that also convolves over the last ``--taps`` rows and norms over
+    turns and stores (``--impl plain``), the one for values that are their keys, without norms and with a bias (``shared``:
+    elements i and i + d / 2 turn together; ``shared-interleaved``: neighbours do), or the one that also convolves over the last ``--taps`` rows and norms over
     the whole projection (``--impl conv``).  ``--tokens`` rows of one request, or ``--batch`` requests of one row
     each.  Bytes: the projection read once (``taps`` times by the convolution, from L2), q, k and v written once."""
     nh, nkv, d, ps = args.heads, args.kv_heads, args.head_dim, args.page_size
@@ -210,7 +226,8 @@ def store(args) -> dict:
     row_request = torch.tensor([r for r, t in enumerate(lens) for _ in range(t)], dtype=torch.int32, device=dev)
     q_start = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
     slots = torch.arange(len(lens), dtype=torch.int32, device=dev)
-    channels = (nh + 2 * nkv) * d
+    shared = args.impl.startswith("shared")
+    channels = (nh + (1 if shared else 2) * nkv) * d
     proj = torch.randn(n, channels, device=dev).to(torch.bfloat16)
     k_pages = torch.zeros(sum(pages_per), nkv, ps, d, device=dev, dtype=torch.bfloat16)
     v_pages = torch.zeros_like(k_pages)
@@ -230,12 +247,17 @@ def store(args) -> dict:
                                          v_pages, q, shift_single=max(lens) == 1)
             if max(lens) > 1:
                 kernels.conv_state_shift(proj, 0, channels, args.taps, state, 0, q_start, slots, len(lens))
+    elif shared:
+        bias = torch.randn(channels, device=dev)
+        fn = lambda: kernels.qk_norm_rope_store(proj, nh, nkv, d, True, None, None, 0.0, cos, sin, d, positions,  # noqa: E731
+                                                row_request, table, k_pages, v_pages, q,
+                                                interleaved=args.impl == "shared-interleaved", bias=bias, value_is_key=True)
     else:
         w = torch.ones(d, device=dev, dtype=torch.bfloat16)
         fn = lambda: kernels.qk_norm_rope_store(proj, nh, nkv, d, True, w, w, 1e-5, cos, sin, d, positions,      # noqa: E731
                                                 row_request, table, k_pages, v_pages, q)
     us = _time(fn, args.iters)
-    byts = 2 * n * channels * 2
+    byts = 2 * n * (channels + (nh + 2 * nkv) * d)
     return {"kernel": f"store/{args.form}/{args.impl}", "heads": nh, "kv_heads": nkv, "head_dim": d, "rows": n,
             "us": round(us, 2), "GBps": round(byts / us / 1e3, 1), "TFLOPs": 0.0}
 
@@ -421,7 +443,9 @@ def latent_store(args) -> dict:
 def residual(args) -> dict:
     """What stands between two sub-layers, for ``tokens`` rows of ``width``.  impl ``sandwich``: the norm and scale on the
     output, the addition, an average over ``planes`` earlier results (0: none), the next norm, and with ``taps`` > 0 (single
-    rows) the convolution; ``streams``: the update, read and norm of two streams in four parts; ``add``: addition and norm.
+    rows) the convolution; ``sum``: addition of an output, a bias and float rows, and norm; ``route``: addition and norm with the
+    choice of ``experts`` experts in four groups; ``add-route``: the same as addition and norm, the router's product and its own
+    kernel; ``streams``: the update, read and norm of two streams in four parts; ``add``: addition and norm.
     Bytes: every float32 and bfloat16 row once each way."""
     n, w, planes = args.tokens, args.width, args.planes
     dev, dtype = torch.device("cuda"), torch.bfloat16
@@ -435,6 +459,24 @@ def residual(args) -> dict:
         x = torch.randn(n, w, device=dev)
         fn = lambda: kernels.add_rms_norm(x, y, weight, 1e-5, out)                                   # noqa: E731
         byts = n * w * (8 + 4)
+    elif args.impl == "sum":
+        x, bias, plus = torch.randn(n, w, device=dev), torch.randn(w, device=dev), torch.randn(n, w, device=dev)
+        fn = lambda: kernels.sum_norm_route(x, y, bias, plus, weight, 1e-5, out)                     # noqa: E731
+        byts = n * w * (8 + 4 + 4)
+    elif args.impl in ("route", "add-route"):
+        experts = args.experts
+        x, shares = torch.randn(n, w, device=dev), torch.empty(n, experts, device=dev)
+        router = kernels.Router(n_experts=experts, top=2, correction=torch.randn(experts, device=dev), groups=4, keep=2,
+                                mode=kernels.ROUTE_SIGMOID_SHARE, weight=(torch.randn(experts, w, device=dev) * 0.02).to(dtype))
+        logits = torch.empty(n, experts, device=dev)
+
+        def separate():
+            kernels.add_rms_norm(x, y, weight, 1e-5, out)
+            kernels.linear(out, router.weight, logits, dtype)
+            kernels.route(logits, router, shares, dtype)
+        fn = separate if args.impl == "add-route" else \
+            (lambda: kernels.sum_norm_route(x, y, None, None, weight, 1e-5, out, router=router, shares=shares))
+        byts = n * w * (8 + 4) + 2 * experts * w + 4 * n * experts
     else:
         x, post = torch.randn(n, w, device=dev), torch.randn(w, device=dev)
         past = torch.randn(planes, n, w, device=dev) if planes else None
@@ -789,7 +831,9 @@ def main(argv=None) -> int:
     a.add_argument("--min-tiles", type=int, default=0, help="decode form: fewest 64-key tiles per slice (0: as the engine chooses)")
     a.add_argument("--max-context", type=int, default=0, help="decode form: the context that the grid is sized for")
     a.add_argument("--window", type=int, default=0, help="a sliding window of that many keys (0: every earlier key)")
-    a.add_argument("--per-head", action="store_true", help="mma: a factor, a slope and a sink per head on the scores")
+    a.add_argument("--per-head", action="store_true", help="a factor, a slope and a sink per head on the scores")
+    a.add_argument("--options", default="", help="further options of the attention: cap, sink, gate, with commas between them")
+    a.add_argument("--keep", type=int, default=0, help="keys at the start of the sequence that are seen beside the window")
     a.add_argument("--heads", type=int, default=32)
     a.add_argument("--kv-heads", type=int, default=8)
     a.add_argument("--head-dim", type=int, default=128)
@@ -811,7 +855,7 @@ def main(argv=None) -> int:
     sc.set_defaults(fn=scan)
     so = sub.add_parser("store")
     so.add_argument("--form", choices=["decode", "prefill"], default="prefill")
-    so.add_argument("--impl", choices=["plain", "conv"], default="conv")
+    so.add_argument("--impl", choices=["plain", "conv", "shared", "shared-interleaved"], default="conv")
     so.add_argument("--batch", type=int, default=8)
     so.add_argument("--context", type=int, default=2048)
     so.add_argument("--tokens", type=int, default=2048)
@@ -864,7 +908,8 @@ def main(argv=None) -> int:
     ls.set_defaults(fn=latent_store)
 
     rs = sub.add_parser("residual")
-    rs.add_argument("--impl", choices=["sandwich", "streams", "add"], default="sandwich")
+    rs.add_argument("--impl", choices=["sandwich", "streams", "add", "sum", "route", "add-route"], default="sandwich")
+    rs.add_argument("--experts", type=int, default=8)
     rs.add_argument("--tokens", type=int, default=2048)
     rs.add_argument("--width", type=int, default=2048)
     rs.add_argument("--planes", type=int, default=0)

@@ -86,7 +86,9 @@ def make_weights(config: dict, seed: int) -> Dict[str, torch.Tensor]:
         elif len(d.shape) == 1:                               # norm weights around one
             t = 1.0 + 0.2 * r
         else:
-            t = r * ((2.0 if n.endswith((".q", ".k", ".router", ".g")) else 1.0) / d.shape[1] ** 0.5)
+            size = 1.3 if n.endswith((".q", ".k")) else 2.0 if n.endswith((".router", ".g")) else \
+                0.6 if n.endswith((".o", ".down")) else 1.0
+            t = r * (size / d.shape[1] ** 0.5)
         out[n] = t.to(torch.bfloat16).to(torch.float32)
     return out
 

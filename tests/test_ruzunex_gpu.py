@@ -770,6 +770,7 @@ def test_attention_with_a_factor_a_slope_and_a_sink_per_head(H, G, D, E, window,
                             token_ids=dev([0] * rows))
         from inferrs_b200.engine.batch import StepContext
         c.attention_tiles = lambda tokens, portions_only=False: StepContext.attention_tiles(c, tokens, portions_only)
+        c.single_rows = lambda: StepContext.single_rows(c)
         return c
 
     out = torch.empty(T, H * E, dtype=dtype, device="cuda")
