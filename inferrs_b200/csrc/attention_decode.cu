@@ -64,7 +64,8 @@ struct Params {
     const int* reqs;           // [R] or null: its request (row of the block table); a negative row is no work
     int max_pages, page_size, n_pages, n_heads, n_kv_heads, window, max_splits, min_tiles;
     float scale_log2;
-    float cap_k, cap_c;        // see ib_capped_log2
+    float slope_factor;        // log2(e); with a cap it and scale_log2 carry ib_cap_factor too (see ib_capped_log2)
+    float cap_c;
     IbScoreOptions opt;
 };
 
@@ -196,7 +197,7 @@ __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constan
                 if (!row_ok[h]) continue;
                 const int head = kvh * G + gid + 8 * h;
                 if (P.opt.head_scale) scale_r[h] *= P.opt.head_scale[head];
-                if (P.opt.slopes) slope_r[h] = P.opt.slopes[head] * 1.4426950408889634f;
+                if (P.opt.slopes) slope_r[h] = P.opt.slopes[head] * P.slope_factor;
             }
         }
         for (int i = 0; i < n_tiles; ++i) {
@@ -230,7 +231,7 @@ __global__ void __launch_bounds__(THREADS, 2) decode_kernel(const __grid_constan
                     float x = sc[n][e] * scale_r[h];
                     if (OPTIONS) {
                         x -= slope_r[h] * (float)(pos - j);
-                        if (P.opt.cap > 0.0f) x = ib_capped_log2(x, P.cap_k, P.cap_c);
+                        if (P.opt.cap > 0.0f) x = ib_capped_log2(x, P.cap_c);
                     }
                     sc[n][e] = vis ? x : -INFINITY;
                     mx[h] = fmaxf(mx[h], sc[n][e]);
@@ -453,7 +454,8 @@ IB_EXPORT int ib_paged_attention_decode(const void* q, const void* k_pages, cons
     P.n_pages = n_pages; P.n_heads = n_heads; P.n_kv_heads = n_kv_heads; P.window = window; P.max_splits = max_splits;
     P.min_tiles = min_tiles;
     P.scale_log2 = scale * 1.4426950408889634f;
-    P.cap_k = cap > 0.0f ? 2.0f / cap : 0.0f;      // the scores carry the factor log2(e) already
+    if (cap > 0.0f) P.scale_log2 *= ib_cap_factor(cap);
+    P.slope_factor = 1.4426950408889634f * (cap > 0.0f ? ib_cap_factor(cap) : 1.0f);
     P.cap_c = cap * 1.4426950408889634f;
     P.opt = {head_scale, slopes, sinks, cap, keep_first, (const act_t*)gate, gate_ld, out_ld};
     const size_t smem = 2 * dec::STAGES * dec::TILE_BYTES + 16 * dec::D * 2 + (2 * dec::STAGES + 1) * 8 + 1024;

@@ -74,7 +74,8 @@ struct AttnMmaParams {
     float* part_ml;                //                          [N, n_heads, splits, 2]
     int max_pages, page_size, n_pages, n_heads, n_kv_heads, window, n_splits;
     float scale_log2;              // scale * log2(e)
-    float cap_k, cap_c;            // see ib_capped_log2
+    float slope_factor;            // log2(e); with a cap it and scale_log2 carry ib_cap_factor too (see ib_capped_log2)
+    float cap_c;
     IbScoreOptions opt;
 };
 
@@ -156,7 +157,7 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
         const int head = kvh * G + (r - ti * G);
         const bool head_ok = r - ti * G < G && head < P.n_heads && (DECODE ? r < G : true);
         scale_r[h] = P.scale_log2 * ((P.opt.head_scale && head_ok) ? P.opt.head_scale[head] : 1.0f);
-        slope_r[h] = (P.opt.slopes && head_ok) ? P.opt.slopes[head] * AM_LOG2E : 0.0f;
+        slope_r[h] = (P.opt.slopes && head_ok) ? P.opt.slopes[head] * P.slope_factor : 0.0f;
         if (ti < n_tok) {
             pos_r[h] = p0 + ti;
             lo_r[h] = ib_first_visible(pos_r[h], P.window);
@@ -228,7 +229,7 @@ __global__ void __launch_bounds__(AM_THREADS) paged_attention_mma_kernel(const A
                 const int j = t * AM_KEYS + col0 + (i & 1);
                 const bool vis = ib_visible(j, lo_r[h], pos_r[h], keep);
                 float x = s[n][i] * scale_r[h] - slope_r[h] * (float)(pos_r[h] - j);
-                if (P.opt.cap > 0.0f) x = ib_capped_log2(x, P.cap_k, P.cap_c);
+                if (P.opt.cap > 0.0f) x = ib_capped_log2(x, P.cap_c);
                 s[n][i] = vis ? x : -INFINITY;
                 mx[h] = fmaxf(mx[h], s[n][i]);
             }
@@ -420,7 +421,8 @@ IB_EXPORT int ib_paged_attention_mma(const void* q, const void* k_pages, const v
     P.max_pages = max_pages; P.page_size = page_size; P.n_pages = n_pages; P.n_heads = n_heads;
     P.n_kv_heads = n_kv_heads; P.window = window; P.n_splits = decode_form ? (n_splits < 1 ? 1 : n_splits) : 1;
     P.scale_log2 = scale * AM_LOG2E;
-    P.cap_k = cap > 0.0f ? 2.0f / cap : 0.0f;      // the scores carry the factor log2(e) already
+    if (cap > 0.0f) P.scale_log2 *= ib_cap_factor(cap);
+    P.slope_factor = AM_LOG2E * (cap > 0.0f ? ib_cap_factor(cap) : 1.0f);
     P.cap_c = cap * AM_LOG2E;
     P.opt = {head_scale, slopes, sinks, cap, keep_first, (const act_t*)gate, gate_ld, out_ld};
     int rc;

@@ -59,7 +59,8 @@ struct Params {
     __nv_bfloat16* out;       // [N, n_heads * 128]
     int max_pages, page_size, n_pages, n_heads, n_kv_heads, window;
     float scale_log2;
-    float cap_k, cap_c;       // see ib_capped_log2
+    float slope_factor;       // log2(e); with a cap it and scale_log2 carry ib_cap_factor too (see ib_capped_log2)
+    float cap_c;
     IbScoreOptions opt;
 };
 
@@ -233,7 +234,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_cons
         if (PER_HEAD && g < G && kvh * G + g < P.n_heads) {
             const int head = kvh * G + g;
             if (P.opt.head_scale) sc2 *= P.opt.head_scale[head];
-            if (P.opt.slopes) sl2 = P.opt.slopes[head] * FA_LOG2E;
+            if (P.opt.slopes) sl2 = P.opt.slopes[head] * P.slope_factor;
             if (P.opt.sinks) sink2 = P.opt.sinks[head] * FA_LOG2E;
         }
         float o[64];
@@ -281,8 +282,8 @@ __global__ void __launch_bounds__(THREADS, 1) attention_kernel(const __grid_cons
                                        ? fmaf(__uint_as_float(b[j]), sc2, fmaf(sl2, (float)(32 + j), base))
                                        : __uint_as_float(b[j]) * sc2;
                         if (CAPPED) {
-                            va = ib_capped_log2(va, P.cap_k, P.cap_c);
-                            vb = ib_capped_log2(vb, P.cap_k, P.cap_c);
+                            va = ib_capped_log2(va, P.cap_c);
+                            vb = ib_capped_log2(vb, P.cap_c);
                         }
                         if (decltype(with_mask)::value) {
                             const int ka = key0 + j, kb = key0 + 32 + j;
@@ -454,7 +455,8 @@ IB_EXPORT int ib_paged_attention_tcgen05(const void* q, const void* k_pages, con
     P.positions = positions; P.out = (__nv_bfloat16*)out; P.max_pages = max_pages; P.page_size = page_size;
     P.n_pages = n_pages; P.n_heads = n_heads; P.n_kv_heads = n_kv_heads; P.window = window;
     P.scale_log2 = scale * FA_LOG2E;
-    P.cap_k = cap > 0.0f ? 2.0f / cap : 0.0f;      // the scores carry the factor log2(e) already
+    if (cap > 0.0f) P.scale_log2 *= ib_cap_factor(cap);
+    P.slope_factor = FA_LOG2E * (cap > 0.0f ? ib_cap_factor(cap) : 1.0f);
     P.cap_c = cap * FA_LOG2E;
     P.opt = {head_scale, slopes, sinks, cap, keep_first, (const act_t*)gate, gate_ld, out_ld};
     const size_t smem = 7 * fa::TILE_BYTES + 18 * 8 + 4 * 128 * 4 + fa::SMEM_SLACK;

@@ -84,11 +84,15 @@ __device__ __forceinline__ float ib_head_gate(const IbScoreOptions& o, long row,
     return o.gate ? 1.0f / (1.0f + expf(-ib_to_float(o.gate[row * o.gate_ld + head]))) : 1.0f;
 }
 
-// The cap for kernels whose scores carry a factor log2(e): cap log2(e) tanh(x / cap) of x = raw * factor, through
-// tanh(y) = 1 - 2 / (1 + e^(2 y)), with k = 2 / cap and c = cap log2(e).  Absolute error about c * 2^-22.
-__device__ __forceinline__ float ib_capped_log2(float x, float k, float c) {
-    const float t = exp2f(x * k);
-    return c - __fdividef(2.0f * c, 1.0f + t);
+// The cap for kernels whose scores carry a factor log2(e): with c = cap log2(e), c tanh(x / c) of a score x, through
+// tanh(z) = 1 - 2 / (1 + 2^(2 z log2(e))); y is x times ib_cap_factor(cap).  Absolute error about c * 2^-22: far below
+// what rounding the keys to bfloat16 does to a score.
+static inline float ib_cap_factor(float cap) { return 2.0f / cap; }      // 2 log2(e) / c
+__device__ __forceinline__ float ib_capped_log2(float y, float c) {
+    float t, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(t) : "f"(y));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + t));         // of infinity: zero
+    return fmaf(-2.0f * c, r, c);
 }
 
 // 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))

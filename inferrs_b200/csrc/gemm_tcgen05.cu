@@ -609,10 +609,24 @@ static int sm_count() {
 // of such a product are made lower than the MMA (which then computes rows that nobody stores) until there are as
 // many CTAs as the GPU holds.  `full` is the MMA's share of rows per tile: 128, or 64 of each matrix in the gated
 // form; `resident` what resident_ctas() says for the kernel that will run.
+//
+// A product of several waves whose last wave would be a handful of CTAs (297 tiles where 296 fit) ends with these alone on
+// the GPU, each at the pace of one CTA's ring: its tiles are made lower until the last wave is two fifths full, which a
+// CTA per SM still streams at the memory's pace.
 static int tile_rows_for(int n_out, int splits, int full, int resident) {
     if (!g_even_tiles || resident <= 0) return full;
     const long ctas_full = (long)((n_out + full - 1) / full) * splits;
-    if (ctas_full > resident || ctas_full <= sm_count()) return full;   // several waves anyway, or one CTA per SM at most   // several waves anyway, or one CTA per SM at most
+    if (ctas_full > resident) {
+        if (splits != 1 || full != tc::BM) return full;
+        const long last = ctas_full % resident;
+        if (last == 0 || 8 * last >= resident) return full;
+        for (int rows = full - 8; rows >= full / 2; rows -= 8) {
+            const long r = ((n_out + rows - 1) / rows) % resident;
+            if (5 * r >= 2 * resident) return rows;
+        }
+        return full;
+    }
+    if (ctas_full <= sm_count()) return full;               // one CTA per SM at most
     const int tiles_wanted = resident / splits;
     int rows = (n_out + tiles_wanted - 1) / tiles_wanted;
     rows = (rows + 7) / 8 * 8;                              // a few CTAs fewer than fit: the next kernel's first ones find room

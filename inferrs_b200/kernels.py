@@ -1446,7 +1446,7 @@ def sum_norm_routes(width: int, router: Router) -> bool:
     """Whether the kernel that norms a row also routes it at these sizes."""
     up4 = lambda v: (v + 3) // 4 * 4                                                              # noqa: E731
     return width <= SUM_NORM_MAX_WIDTH and router.n_experts <= 2048 and \
-        4 * (up4(width) + up4(router.columns) + 5 * router.n_experts) <= SUM_NORM_MAX_SHARED
+        4 * (2 * up4(width) + up4(router.columns) + 5 * router.n_experts) <= SUM_NORM_MAX_SHARED
 
 
 def sum_norm_route(residual: torch.Tensor, delta: Optional[torch.Tensor], bias: Optional[torch.Tensor],

@@ -89,7 +89,9 @@ class Dense:
 register_feed_forward("dense", Dense)
 
 
-ROUTER_BESIDE_NORM_BYTES = 64 << 20     # what the rows' blocks may read of a router matrix from L2, all together
+# a norm kernel makes router logits of up to so many rows, and with matrices of up to so many bytes: beyond, a product of its
+# own is faster (measured at 8 and 64 experts)
+ROUTER_BESIDE_NORM_ROWS, ROUTER_BESIDE_NORM_BYTES = 64, 256 << 10
 
 
 class RoutedExperts:
@@ -190,7 +192,7 @@ class RoutedExperts:
         """The router for a norm kernel that makes its logits too; None where a product of its own is better (many
         rows: every row's block reads the whole matrix)."""
         w = self.router.weight
-        fits = n_rows * w.numel() * w.element_size() <= ROUTER_BESIDE_NORM_BYTES
+        fits = n_rows <= ROUTER_BESIDE_NORM_ROWS and w.numel() * w.element_size() <= ROUTER_BESIDE_NORM_BYTES
         return self.routing if fits and kernels.sum_norm_routes(self.spec.width, self.routing) else None
 
     def middle(self, ctx, cache_id, h, proj: torch.Tensor, out: torch.Tensor, shares=None):
