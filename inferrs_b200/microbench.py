@@ -491,8 +491,9 @@ def residual(args) -> dict:
                                            result=res, conv=conv)
         byts = n * w * (8 + 4 + (planes + 1) * 4 * bool(planes) + 8 * max(args.taps - 1, 0))
     us = _time(fn, args.iters)
-    return {"kernel": f"residual/{args.impl}", "rows": n, "width": w, "planes": planes, "taps": args.taps, "us": round(us, 2),
-            "GBps": round(byts / us / 1e3, 1), "TFLOPs": 0.0}
+    return dict({"kernel": f"residual/{args.impl}", "rows": n, "width": w, "planes": planes, "taps": args.taps, "us": round(us, 2),
+                 "GBps": round(byts / us / 1e3, 1), "TFLOPs": 0.0},
+                **({"experts": args.experts} if args.impl in ("route", "add-route") else {}))
 
 
 def activation(args) -> dict:
